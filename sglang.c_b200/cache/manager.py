@@ -31,7 +31,9 @@ class _Group:
 class CacheManager:
     """needs[i] is the CacheNeed (or None) of the i-th call of the running
     order; cache_of[i] names the earlier call whose cache call i reads.
-    A need may be a tuple of needs; the call's binding is then a tuple of bindings.
+    A need may be a tuple of needs; the call's binding is then a tuple of bindings.  A call that
+    reads another's cache reads the needs that are not private, matched in order; private ones it
+    keeps for itself.
     `make_tensor(shape, dtype_name)` allocates device memory (None in host-only
     tests)."""
 
@@ -54,9 +56,9 @@ class CacheManager:
                 return []
             return list(enumerate(need)) if isinstance(need, (tuple, list)) else [(None, need)]
         for i in range(len(needs)):
-            if cache_of[i] is not None:
-                continue
             for j, need in subs(i):
+                if cache_of[i] is not None and not need.private:
+                    continue
                 gi = by_need.get(need)
                 if gi is None:
                     gi = len(self.groups)
@@ -85,15 +87,20 @@ class CacheManager:
             if needs[i] is None:
                 continue
             owner = i if cache_of[i] is None else cache_of[i]
-            if needs[owner] != needs[i]:
+            shared = [(j, need) for j, need in subs(owner) if not need.private]
+            if [need for _, need in shared] != [need for _, need in subs(i) if not need.private]:
                 raise CacheError(f"call {i} reads the cache of call {owner} but their needs differ")
-            made = []
+            made, k = [], 0
             for j, need in subs(i):
-                if (owner, j) not in self._call_group:
+                at = (i, j)
+                if not need.private:
+                    at = (owner, shared[k][0])
+                    k += 1
+                if at not in self._call_group:
                     raise CacheError(f"call {i} reads the cache of call {owner}, which keeps none")
-                gi, ci = self._call_group[(owner, j)]
+                gi, ci = self._call_group[at]
                 t = self.groups[gi].tensor
-                made.append(CacheBinding(need.kind, gi, t[ci] if t is not None else None, write=(owner == i)))
+                made.append(CacheBinding(need.kind, gi, t[ci] if t is not None else None, write=(at[0] == i)))
             self._bindings[i] = tuple(made) if isinstance(needs[i], (tuple, list)) else made[0]
         # per-request bookkeeping
         self._free_slots = list(range(self.max_requests - 1, -1, -1))

@@ -14,8 +14,9 @@ class CacheNeed:
     keys' `head_dim`; a page is then one flat block, n_kv_heads x page_size x head_dim keys followed
     by n_kv_heads x page_size x v_dim values.  `chunk` (paged_kv): a query sees only keys of its own
     chunk of so many positions (counted from position 0), so pages of earlier chunks go back to the
-    pool as a window's do.  A mixer with several things to keep answers with a tuple of needs and
-    gets a tuple of bindings."""
+    pool as a window's do.  `private` (state): a call that reads another call's cache still keeps this
+    one for itself (the tail of a convolution over its own queries, beside another call's keys).
+    A mixer with several things to keep answers with a tuple of needs and gets a tuple of bindings."""
     kind: str
     n_kv_heads: int = 0
     head_dim: int = 0
@@ -25,6 +26,7 @@ class CacheNeed:
     shared: bool = False
     v_dim: Optional[int] = None
     chunk: Optional[int] = None
+    private: bool = False
 
     @classmethod
     def paged_kv(cls, n_kv_heads, head_dim, window=None, shared=False, v_dim=None, chunk=None):
@@ -39,8 +41,8 @@ class CacheNeed:
                    chunk=None if chunk is None else int(chunk))
 
     @classmethod
-    def state(cls, shape, dtype="float32"):
-        return cls("state", state_shape=tuple(int(s) for s in shape), state_dtype=dtype)
+    def state(cls, shape, dtype="float32", private=False):
+        return cls("state", state_shape=tuple(int(s) for s in shape), state_dtype=dtype, private=bool(private))
 
 
 @dataclass

@@ -12,6 +12,9 @@
 //   values   a thread two adjacent columns of some heads' results: acc = acc * corr + sum_j p_j c_j
 // With one range the result is normalised and written; with several, every range leaves
 // (m, l, acc) in a workspace and a second small launch merges them in range order.
+// Whoever writes the result also lets a sink per head join the softmax's denominator (a learned
+// score with no row and no value, unscaled, counted once) and multiplies a head's result by the sigmoid
+// of a number per head or per entry, where the caller gives them.
 #include "common.cuh"
 
 SGLC_DEFINE_ERROR_STRING()
@@ -39,7 +42,15 @@ struct LatentArgs {
   float scale;
   float* ws;                 // [T][n_splits][H][D + 2] when n_splits > 1
   int* err;
+  const float* sinks;        // [H] or null
+  const float* gate;         // pre-activations, rows gate_stride apart, or null
+  long long gate_stride;
+  int gate_per_head;         // 1: gate[t][h]; 0: gate[t][h * D + d]
 };
+
+__device__ __forceinline__ float gate_of(const LatentArgs& a, int t, int h, int d) {
+  return 1.0f / (1.0f + expf(-a.gate[(size_t)t * a.gate_stride + (a.gate_per_head ? h : h * a.D + d)]));
+}
 
 __global__ void __launch_bounds__(THREADS)
 latent_decode_kernel(LatentArgs a) {
@@ -162,8 +173,18 @@ latent_decode_kernel(LatentArgs a) {
     for (int i = 0; i < MAX_ACC; i++) {
       const int pair = i * THREADS + tid;
       if (pair < n_pairs) {
-        const float inv = 1.0f / l_s[(2 * pair) / D];
-        *reinterpret_cast<__nv_bfloat162*>(op + 2 * pair) = __floats2bfloat162_rn(acc[i].x * inv, acc[i].y * inv);
+        const int h = (2 * pair) / D, d = (2 * pair) % D;
+        float inv = 1.0f / l_s[h];
+        if (a.sinks) {
+          const float sk = a.sinks[h0 + h], top = fmaxf(m_s[h], sk), keep = expf(m_s[h] - top);
+          inv = keep / (l_s[h] * keep + expf(sk - top));
+        }
+        float y0 = acc[i].x * inv, y1 = acc[i].y * inv;
+        if (a.gate) {
+          y0 *= gate_of(a, t, h0 + h, d);
+          y1 *= gate_of(a, t, h0 + h, d + 1);
+        }
+        *reinterpret_cast<__nv_bfloat162*>(op + 2 * pair) = __floats2bfloat162_rn(y0, y1);
       }
     }
     return;
@@ -207,17 +228,19 @@ latent_merge_kernel(LatentArgs a) {
     l[sp] = on ? w[sp * step + D + 1] : 0.0f;
     v[sp] = on ? w[sp * step + d] : 0.0f;
   }
-  float M = -INFINITY;
+  float M = a.sinks ? a.sinks[h] : -INFINITY;
 #pragma unroll
   for (int sp = 0; sp < MAX_SPLITS; sp++) M = fmaxf(M, m[sp]);
-  float L = 0.0f, o = 0.0f;
+  float L = a.sinks ? expf(a.sinks[h] - M) : 0.0f, o = 0.0f;
 #pragma unroll
   for (int sp = 0; sp < MAX_SPLITS; sp++) {
     const float f = l[sp] > 0.0f ? expf(m[sp] - M) : 0.0f;      // (a range past the token's keys is empty)
     L = fmaf(l[sp], f, L);
     o = fmaf(v[sp], f, o);
   }
-  a.out[(size_t)t * a.o_stride + i] = __float2bfloat16_rn(o / L);
+  o /= L;
+  if (a.gate) o *= gate_of(a, t, h, d);
+  a.out[(size_t)t * a.o_stride + i] = __float2bfloat16_rn(o);
 }
 }  // namespace
 
@@ -243,12 +266,14 @@ SGLC_API int sglc_attention_latent_decode_splits(int T, int max_keys) {
 // q, out: bfloat16 [T][stride], heads side by side (H * D columns); cache: bfloat16 rows
 // [n_pages][page_size][D]; positions[t]: the token's own position (its row is in the cache);
 // T: tokens this launch serves (all, or the first T of token_list); ws: n_splits > 1 needs
-// T * n_splits * H * (D + 2) floats.
+// T * n_splits * H * (D + 2) floats; sinks: float [H] or null; gate: float rows gate_stride apart, or null.
 SGLC_API int sglc_attention_latent_decode(const void* q, int q_stride, const void* cache, const int* block_table,
                                           int bt_stride, const int* token_req, const int* positions,
                                           const int* token_list, void* out, int o_stride, int T, int H, int D,
                                           int page_size, float scale, int window, int n_splits, float* ws,
-                                          long long ws_floats, int n_pages, int* err, cudaStream_t stream) {
+                                          long long ws_floats, int n_pages, int* err, const float* sinks,
+                                          const float* gate, long long gate_stride, int gate_per_head,
+                                          cudaStream_t stream) {
   if (T <= 0) return SGLC_OK;
   if (page_size <= 0 || n_splits < 1) return SGLC_ERR_ARGUMENT;
   if (!sglc_attention_latent_decode_supports(H, D) || n_splits > MAX_SPLITS) return SGLC_ERR_UNSUPPORTED;
@@ -262,6 +287,7 @@ SGLC_API int sglc_attention_latent_decode(const void* q, int q_stride, const voi
   a.out = (__nv_bfloat16*)out; a.o_stride = o_stride;
   a.H = H; a.D = D; a.page_size = page_size; a.window = window; a.n_splits = n_splits; a.n_pages = n_pages;
   a.scale = scale; a.ws = ws; a.err = err;
+  a.sinks = sinks; a.gate = gate; a.gate_stride = gate_stride; a.gate_per_head = gate_per_head;
   // heads are dealt to several blocks while the launch has fewer than one and a half blocks an SM
   const long long base = (long long)T * n_splits;
   int groups = (int)((222 + base - 1) / base);

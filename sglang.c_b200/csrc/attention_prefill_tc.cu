@@ -64,6 +64,9 @@ struct Args {
   int kv_shared;          // pages [1][Hkv][page_size][D]: one block of rows serves as keys and as values
   int chunk;              // > 0: a query sees only the keys of its own chunk of so many positions (counted from 0)
   const float* sinks;     // [H] or null: a score per head that joins the softmax's denominator once, unscaled
+  const float* gate;      // null, or pre-activations whose sigmoid multiplies the heads' results: [T][gate_stride],
+  long long gate_stride;  //   one number per head (gate_per_head) or one per entry (h * D + d)
+  int gate_per_head;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
@@ -86,8 +89,8 @@ __device__ __forceinline__ float ex2_approx(float x) {
 // byte offset of 16-byte chunk `c` (0..7) of row `r` in a [rows][128 B] tile with the 128-byte swizzle
 __device__ __forceinline__ uint32_t sw128(int r, int c) { return (uint32_t)(r * 128 + ((c ^ (r & 7)) << 4)); }
 
-// EXT: the instantiation that also knows a chunk mask and sinks (Args::chunk, Args::sinks); the
-// plain one is compiled without either.
+// EXT: the instantiation that also knows a chunk mask, sinks and an output gate (Args::chunk, sinks,
+// gate); the plain one is compiled without them.
 template <int D, bool EXT>
 __global__ void __launch_bounds__(THREADS, (D == 64 ? 2 : 1))
 attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
@@ -575,11 +578,26 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q,
           const float keep = exp2f(ms - top);
           inv = keep / (l[x] * keep + exp2f(sk - top));
         }
+        const float* gz = nullptr;
+        if (EXT && a.gate) {
+          gz = a.gate + (size_t)(t0 + qt * BQ + row_r[x]) * a.gate_stride;
+          if (a.gate_per_head) {
+            inv *= 1.0f / (1.0f + expf(-gz[h]));
+            gz = nullptr;
+          } else {
+            gz += (size_t)h * D + 2 * q4;
+          }
+        }
         __nv_bfloat16* op = a.out + (size_t)(t0 + qt * BQ + row_r[x]) * a.o_stride + (size_t)h * D + 2 * q4;
 #pragma unroll
         for (int i = 0; i < D / 8; i++) {          // the row's i-th block of 8 columns
           if (i < keep0 || i >= keep0 + n_keep) continue;
-          __nv_bfloat162 hh = __floats2bfloat162_rn(o[4 * i + 2 * x] * inv, o[4 * i + 2 * x + 1] * inv);
+          float y0 = o[4 * i + 2 * x] * inv, y1 = o[4 * i + 2 * x + 1] * inv;
+          if (EXT && gz) {
+            y0 *= 1.0f / (1.0f + expf(-gz[8 * i]));
+            y1 *= 1.0f / (1.0f + expf(-gz[8 * i + 1]));
+          }
+          __nv_bfloat162 hh = __floats2bfloat162_rn(y0, y1);
           *reinterpret_cast<__nv_bfloat162*>(op + 8 * i) = hh;
         }
       }
@@ -685,7 +703,8 @@ static int attention_prefill_run(const void* q, int q_stride, const void* cache,
                                  int max_q_len, int H, int Hkv, int D, int page_size,
                                  float scale, int window, int T, int n_pages, int skip_single,
                                  int* err, int kv_shared, cudaStream_t stream, int chunk = 0,
-                                 const float* sinks = nullptr) {
+                                 const float* sinks = nullptr, const float* gate = nullptr,
+                                 long long gate_stride = 0, int gate_per_head = 0) {
   if (R <= 0 || max_q_len <= 0) return SGLC_OK;
   if (chunk < 0) return SGLC_ERR_ARGUMENT;
   if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || page_size <= 0) return SGLC_ERR_ARGUMENT;
@@ -708,6 +727,7 @@ static int attention_prefill_run(const void* q, int q_stride, const void* cache,
   a.kv_shared = kv_shared;
   a.chunk = chunk;
   a.sinks = sinks;
+  a.gate = gate; a.gate_stride = gate_stride; a.gate_per_head = gate_per_head;
   // TMA needs whole pages inside a 128-key tile and rows it can address
   CUtensorMap mq, mkv;
   memset(&mq, 0, sizeof(mq));
@@ -718,7 +738,7 @@ static int attention_prefill_run(const void* q, int q_stride, const void* cache,
               get_kv_map(&mkv, cache, D, page_size, Hkv, n_pages, kv_shared ? 1 : 2);
     a.use_tma = ok ? 1 : 0;
   }
-  if (chunk > 0 || sinks) {
+  if (chunk > 0 || sinks || gate) {
     if (D == 64) return launch<64, true>(mq, mkv, a, R, max_q_len, stream);
     return launch<128, true>(mq, mkv, a, R, max_q_len, stream);
   }
@@ -751,15 +771,18 @@ SGLC_API int sglc_attention_prefill_tc_shared(const void* q, int q_stride, const
 }
 
 // The same with a chunk mask (chunk > 0: a query sees only the keys of its own chunk of so many
-// positions, counted from position 0) and a sink per head (sinks: float [H] or null) in the
-// softmax's denominator.
+// positions, counted from position 0), a sink per head (sinks: float [H] or null) in the softmax's
+// denominator, and a gate (float pre-activations, rows gate_stride apart, or null) whose sigmoid
+// multiplies the heads' results: one number per head (gate_per_head) or one per entry.  kv_shared as
+// in the form above it.
 SGLC_API int sglc_attention_prefill_tc_ext(const void* q, int q_stride, const void* cache,
                                            const int* block_table, int bt_stride, const int* q_start,
                                            const int* kv_len, void* out, int o_stride, int R,
                                            int max_q_len, int H, int Hkv, int D, int page_size,
                                            float scale, int window, int chunk, const float* sinks, int T,
-                                           int n_pages, int skip_single, int* err, cudaStream_t stream) {
+                                           int n_pages, int skip_single, int* err, int kv_shared, const float* gate,
+                                           long long gate_stride, int gate_per_head, cudaStream_t stream) {
   return attention_prefill_run(q, q_stride, cache, block_table, bt_stride, q_start, kv_len, out, o_stride, R,
-                               max_q_len, H, Hkv, D, page_size, scale, window, T, n_pages, skip_single, err, 0,
-                               stream, chunk, sinks);
+                               max_q_len, H, Hkv, D, page_size, scale, window, T, n_pages, skip_single, err, kv_shared,
+                               stream, chunk, sinks, gate, gate_stride, gate_per_head);
 }

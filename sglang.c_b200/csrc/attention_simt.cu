@@ -33,16 +33,28 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float* v) {
 // EXT: the form with a value size DV of its own (a page then holds Hkv x page_size x D keys
 // followed by Hkv x page_size x DV values), a chunk mask (a query sees only keys of its own chunk of
 // `chunk` positions, counted from position 0) and a sink per head (a learned score that joins the
-// softmax's denominator once, with no key and no value).  Without EXT the three arguments are unused.
-template <typename TQ, typename TC, typename TO, int W, int THREADS, bool EXT>
-__global__ void __launch_bounds__(THREADS, THREADS == 256 ? 3 : 4)     // (registers capped so that three blocks of 256 share an SM)
+// softmax's denominator once, with no key and no value), and an output gate (a head's result times
+// the sigmoid of a number per head, or of one per entry).  Without EXT these arguments are unused.
+// NA: columns of the output a lane holds (a head's value size is at most 32 * NA).
+struct OutGate {
+  const float* z;                 // pre-activations, rows `stride` apart (null: no gate)
+  long long stride;
+  int per_head;                   // 1: z[t][h]; 0: z[t][h * DV + d]
+};
+__device__ __forceinline__ float out_gate(const OutGate& g, long long t, int h, int DV, int d) {
+  const float z = g.z[t * g.stride + (g.per_head ? h : h * DV + d)];
+  return 1.0f / (1.0f + expf(-z));
+}
+
+template <typename TQ, typename TC, typename TO, int W, int THREADS, bool EXT, int NA>
+__global__ void __launch_bounds__(THREADS, NA > 8 ? 1 : THREADS == 256 ? 3 : 4)     // (registers capped so that three blocks of 256 share an SM)
 attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restrict__ cache,
                       const int* __restrict__ block_table, int bt_stride,
                       const int* __restrict__ token_req, const int* __restrict__ positions,
                       TO* __restrict__ out, int o_stride, int T, int H, int Hkv, int D, int page_size,
                       float scale, int window, int n_pages, int* err, int kv_shared,
                       int DV_arg, int chunk, const float* __restrict__ sinks, int n_splits,
-                      float* __restrict__ part_ws, int head_rows) {
+                      float* __restrict__ part_ws, int head_rows, const OutGate gate) {
   const int DV = EXT ? DV_arg : D;
   // head_rows (EXT, a step of single tokens): the block's warps are the query heads that share one
   // key/value head, all of ONE token (blockIdx.x), instead of consecutive tokens of one head: the
@@ -81,11 +93,11 @@ attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restri
   __syncthreads();
   const int my_req = mine ? s_req[warp] : -2, my_lo = mine ? s_lo[warp] : 0, my_pos = mine ? s_pos[warp] : -1;
   float m = -INFINITY, l = 0.0f;
-  float acc[8];                               // dims lane, lane + 32, ... of the output
+  float acc[NA];                              // dims lane, lane + 32, ... of the output
 #pragma unroll
-  for (int i = 0; i < 8; i++) acc[i] = 0.0f;
+  for (int i = 0; i < NA; i++) acc[i] = 0.0f;
   // kv_shared: a page holds one block of rows that are keys and values at once (a latent)
-  const size_t page_elems = EXT ? (size_t)Hkv * page_size * (D + DV) : (size_t)(kv_shared ? 1 : 2) * Hkv * page_size * D;
+  const size_t page_elems = EXT && !kv_shared ? (size_t)Hkv * page_size * (D + DV) : (size_t)(kv_shared ? 1 : 2) * Hkv * page_size * D;
   const size_t head_off = (size_t)hk * page_size * D, v_off = kv_shared ? 0 : (size_t)Hkv * page_size * D;
 
   // The tokens of a block that belong to one request (a run: a request's tokens lie together)
@@ -122,7 +134,7 @@ attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restri
             kp = cache + (size_t)page * page_elems + head_off + (size_t)(p % page_size) * D;
         }
         if (EXT) {
-          const TC* vp = kp ? cache + (size_t)(bt[p / page_size]) * page_elems + (size_t)Hkv * page_size * D +
+          const TC* vp = kp && kv_shared ? kp : kp ? cache + (size_t)(bt[p / page_size]) * page_elems + (size_t)Hkv * page_size * D +
                                   ((size_t)hk * page_size + p % page_size) * DV
                             : nullptr;
           if (D % 4 == 0 && DV % 4 == 0) {      // (rows, pages and both blocks of a page start at multiples of four)
@@ -192,7 +204,7 @@ attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restri
           pj[j] = p4.x; pj[j + 1] = p4.y; pj[j + 2] = p4.z; pj[j + 3] = p4.w;
         }
 #pragma unroll
-        for (int i = 0; i < 8; i++) {
+        for (int i = 0; i < NA; i++) {
           const int d = lane + 32 * i;
           if (d < DV) {
             float a = acc[i] * corr;
@@ -211,7 +223,7 @@ attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restri
       float* rec = part_ws + (((size_t)my_t * H + h) * n_splits + blockIdx.z) * (DV + 2);
       if (lane == 0) { rec[0] = m; rec[1] = l; }
 #pragma unroll
-      for (int i = 0; i < 8; i++) {
+      for (int i = 0; i < NA; i++) {
         const int d = lane + 32 * i;
         if (d < DV) rec[2 + d] = acc[i];
       }
@@ -225,10 +237,11 @@ attention_simt_kernel(const TQ* __restrict__ q, int q_stride, const TC* __restri
       const float sk = sinks[h], m_all = fmaxf(m, sk);
       inv = expf(m - m_all) / (l * expf(m - m_all) + expf(sk - m_all));
     }
+    const bool gated = EXT && gate.z;
 #pragma unroll
-    for (int i = 0; i < 8; i++) {
+    for (int i = 0; i < NA; i++) {
       const int d = lane + 32 * i;
-      if (d < DV) op[d] = from_f32<TO>(acc[i] * inv);
+      if (d < DV) op[d] = from_f32<TO>(gated ? acc[i] * inv * out_gate(gate, my_t, h, DV, d) : acc[i] * inv);
     }
   }
 }
@@ -246,55 +259,67 @@ static int attention_simt_run(const void* q, int q_stride, const void* cache,
                               int Hkv, int D, int page_size, float scale, int window,
                               int max_keys, int act_dtype, int cache_dtype, int n_pages, int* err,
                               int max_q_len, int kv_shared, cudaStream_t stream, bool ext = false, int DV = 0,
-                              int chunk = 0, const float* sinks = nullptr, int n_splits = 1, float* part_ws = nullptr) {
+                              int chunk = 0, const float* sinks = nullptr, int n_splits = 1, float* part_ws = nullptr,
+                              OutGate gate = OutGate{nullptr, 0, 0}) {
   if (T <= 0) return SGLC_OK;
   if (!ext) DV = D;
-  if (DV <= 0 || DV > 256 || chunk < 0) return ext ? SGLC_ERR_UNSUPPORTED : SGLC_ERR_ARGUMENT;
+  if (DV <= 0 || chunk < 0 || (kv_shared && DV > D)) return SGLC_ERR_ARGUMENT;
+  if (DV > (ext ? 768 : 256)) return SGLC_ERR_UNSUPPORTED;
   if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || D <= 0 || page_size <= 0 || max_keys <= 0)
     return SGLC_ERR_ARGUMENT;
-  if (H > 65535 || D > 256) return SGLC_ERR_UNSUPPORTED;
+  if (H > 65535 || D > (ext ? 768 : 256)) return SGLC_ERR_UNSUPPORTED;
   // single tokens of many requests share nothing: a token a block; portions: eight tokens a block
   const bool single = max_q_len <= 1;
   const int W = single ? 1 : 8;
   const size_t smem = ((size_t)32 * (D % 4 == 0 ? D + 4 : D + 1) + (size_t)32 * DV + (size_t)W * D + (size_t)W * 32) * sizeof(float);
+  if (smem > 224 * 1024) return SGLC_ERR_UNSUPPORTED;
   if (part_ws && (!ext || !single || n_splits < 1 || n_splits > 65535)) return SGLC_ERR_ARGUMENT;
   dim3 grid((T + W - 1) / W, H, part_ws ? n_splits : 1);
   // single tokens whose shares are merged afterwards: where 2 to 8 query heads share a key/value
   // head, a block takes them all (the eight-warp form, its warps being heads of one token)
-  const int head_rows = (part_ws && H / Hkv >= 2 && H / Hkv <= 8) ? 1 : 0;
+  int head_rows = (part_ws && H / Hkv >= 2 && H / Hkv <= 8) ? 1 : 0;
   const size_t smem_rows = ((size_t)32 * (D % 4 == 0 ? D + 4 : D + 1) + (size_t)32 * DV + (size_t)8 * D + (size_t)8 * 32) * sizeof(float);
+  if (smem_rows > 224 * 1024) head_rows = 0;
+  const bool wide_v = DV > 256;
   if (head_rows) {
     const dim3 grid_rows(T, Hkv, n_splits);
-#define LAUNCH_R(TQ, TC, TO)                                                                            \
+#define LAUNCH_RN(TQ, TC, TO, NA)                                                                      \
   do {                                                                                                 \
     if (smem_rows > 48 * 1024)                                                                         \
-      cudaFuncSetAttribute(attention_simt_kernel<TQ, TC, TO, 8, 256, true>,                            \
+      cudaFuncSetAttribute(attention_simt_kernel<TQ, TC, TO, 8, 256, true, NA>,                        \
                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_rows);               \
-    attention_simt_kernel<TQ, TC, TO, 8, 256, true><<<grid_rows, 256, smem_rows, stream>>>(            \
+    attention_simt_kernel<TQ, TC, TO, 8, 256, true, NA><<<grid_rows, 256, smem_rows, stream>>>(        \
         (const TQ*)q, q_stride, (const TC*)cache, block_table, bt_stride, token_req, positions,        \
         (TO*)out, o_stride, T, H, Hkv, D, page_size, scale, window, n_pages, err, kv_shared, DV,       \
-        chunk, sinks, n_splits, part_ws, 1);                                                           \
+        chunk, sinks, n_splits, part_ws, 1, gate);                                                     \
+  } while (0)
+#define LAUNCH_R(TQ, TC, TO)                                                                           \
+  do {                                                                                                 \
+    if (wide_v) LAUNCH_RN(TQ, TC, TO, 24);                                                             \
+    else LAUNCH_RN(TQ, TC, TO, 8);                                                                     \
   } while (0)
     if (act_dtype == SGLC_F32 && cache_dtype == SGLC_F32) LAUNCH_R(float, float, float);
     else if (act_dtype == SGLC_BF16 && cache_dtype == SGLC_BF16) LAUNCH_R(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
     else return SGLC_ERR_ARGUMENT;
 #undef LAUNCH_R
+#undef LAUNCH_RN
     return sglc_launch_status();
   }
-#define LAUNCH_E(TQ, TC, TO, WW, TH, EX)                                                               \
+#define LAUNCH_E(TQ, TC, TO, WW, TH, EX, NA)                                                           \
   do {                                                                                                 \
     if (smem > 48 * 1024)                                                                              \
-      cudaFuncSetAttribute(attention_simt_kernel<TQ, TC, TO, WW, TH, EX>,                              \
+      cudaFuncSetAttribute(attention_simt_kernel<TQ, TC, TO, WW, TH, EX, NA>,                          \
                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
-    attention_simt_kernel<TQ, TC, TO, WW, TH, EX><<<grid, TH, smem, stream>>>(                          \
+    attention_simt_kernel<TQ, TC, TO, WW, TH, EX, NA><<<grid, TH, smem, stream>>>(                      \
         (const TQ*)q, q_stride, (const TC*)cache, block_table, bt_stride, token_req, positions,        \
         (TO*)out, o_stride, T, H, Hkv, D, page_size, scale, window, n_pages, err, kv_shared, DV,       \
-        chunk, sinks, n_splits, part_ws, 0);                                                           \
+        chunk, sinks, n_splits, part_ws, 0, gate);                                                     \
   } while (0)
 #define LAUNCH(TQ, TC, TO, WW, TH)                                                                     \
   do {                                                                                                 \
-    if (ext) LAUNCH_E(TQ, TC, TO, WW, TH, true);                                                       \
-    else LAUNCH_E(TQ, TC, TO, WW, TH, false);                                                          \
+    if (ext && wide_v) LAUNCH_E(TQ, TC, TO, WW, TH, true, 24);                                         \
+    else if (ext) LAUNCH_E(TQ, TC, TO, WW, TH, true, 8);                                               \
+    else LAUNCH_E(TQ, TC, TO, WW, TH, false, 8);                                                       \
   } while (0)
   if (act_dtype == SGLC_F32 && cache_dtype == SGLC_F32) {
     if (single) LAUNCH(float, float, float, 1, 128);
@@ -338,15 +363,20 @@ SGLC_API int sglc_attention_simt_shared(const void* q, int q_stride, const void*
 // Hkv x page_size x DV values]; out rows hold H heads of DV), `chunk` > 0: a query sees the keys of its
 // own chunk of so many positions only; `sinks` (float [H] or null): a score per head that joins the
 // softmax's denominator.
+// kv_shared: the cache's pages hold one block of rows [Hkv][page_size][D] that are keys, and whose first
+// DV entries are values.  gate (float, rows gate_stride apart, or null): the heads' results are
+// multiplied by its sigmoid, one number per head (gate_per_head) or one per entry.
 SGLC_API int sglc_attention_simt_ext(const void* q, int q_stride, const void* cache,
                                      const int* block_table, int bt_stride, const int* token_req,
                                      const int* positions, void* out, int o_stride, int T, int H,
                                      int Hkv, int D, int DV, int page_size, float scale, int window, int chunk,
                                      const float* sinks, int max_keys, int act_dtype, int cache_dtype, int n_pages,
-                                     int* err, int max_q_len, cudaStream_t stream) {
+                                     int* err, int max_q_len, int kv_shared, const float* gate, long long gate_stride,
+                                     int gate_per_head, cudaStream_t stream) {
   return attention_simt_run(q, q_stride, cache, block_table, bt_stride, token_req, positions, out, o_stride,
                             T, H, Hkv, D, page_size, scale, window, max_keys, act_dtype, cache_dtype,
-                            n_pages, err, max_q_len, 0, stream, true, DV, chunk, sinks);
+                            n_pages, err, max_q_len, kv_shared, stream, true, DV, chunk, sinks, 1, nullptr,
+                            OutGate{gate, gate_stride, gate_per_head});
 }
 
 // The merge behind a launch that dealt a token's keys to several blocks (a step of single tokens):
@@ -355,7 +385,7 @@ SGLC_API int sglc_attention_simt_ext(const void* q, int q_stride, const void* ca
 template <typename TO>
 __global__ void __launch_bounds__(128)
 attention_merge_kernel(const float* __restrict__ part_ws, int n_splits, const float* __restrict__ sinks,
-                       TO* __restrict__ out, int o_stride, int T, int H, int DV) {
+                       TO* __restrict__ out, int o_stride, int T, int H, int DV, const OutGate gate) {
   pdl_launch_dependents();
   const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -377,7 +407,9 @@ attention_merge_kernel(const float* __restrict__ part_ws, int n_splits, const fl
     float o = 0.0f;
     for (int s = 0; s < n_splits; s++)
       if (rec[(size_t)s * (DV + 2) + 1] > 0.0f) o += rec[(size_t)s * (DV + 2) + 2 + d] * expf(rec[(size_t)s * (DV + 2)] - M);
-    op[d] = from_f32<TO>(o * inv);
+    o *= inv;
+    if (gate.z) o *= out_gate(gate, t, h, DV, d);
+    op[d] = from_f32<TO>(o);
   }
 }
 
@@ -388,17 +420,20 @@ SGLC_API int sglc_attention_simt_ext_split(const void* q, int q_stride, const vo
                                            const int* positions, void* out, int o_stride, int T, int H,
                                            int Hkv, int D, int DV, int page_size, float scale, int window, int chunk,
                                            const float* sinks, int max_keys, int act_dtype, int cache_dtype,
-                                           int n_pages, int* err, int n_splits, float* part_ws, cudaStream_t stream) {
+                                           int n_pages, int* err, int kv_shared, const float* gate,
+                                           long long gate_stride, int gate_per_head, int n_splits, float* part_ws,
+                                           cudaStream_t stream) {
   if (T <= 0) return SGLC_OK;
   if (!part_ws || n_splits < 1) return SGLC_ERR_ARGUMENT;
   const int code = attention_simt_run(q, q_stride, cache, block_table, bt_stride, token_req, positions, out, o_stride,
                                       T, H, Hkv, D, page_size, scale, window, max_keys, act_dtype, cache_dtype,
-                                      n_pages, err, 1, 0, stream, true, DV, chunk, nullptr, n_splits, part_ws);
+                                      n_pages, err, 1, kv_shared, stream, true, DV, chunk, nullptr, n_splits, part_ws);
   if (code != SGLC_OK) return code;
   const dim3 grid((unsigned)(((long long)T * H + 3) / 4));
+  const OutGate g{gate, gate_stride, gate_per_head};
   if (act_dtype == SGLC_F32)
     return sglc_launch(attention_merge_kernel<float>, grid, dim3(128), 0, stream, 1, true, (const float*)part_ws,
-                       n_splits, sinks, (float*)out, o_stride, T, H, DV);
+                       n_splits, sinks, (float*)out, o_stride, T, H, DV, g);
   return sglc_launch(attention_merge_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, 1, true,
-                     (const float*)part_ws, n_splits, sinks, (__nv_bfloat16*)out, o_stride, T, H, DV);
+                     (const float*)part_ws, n_splits, sinks, (__nv_bfloat16*)out, o_stride, T, H, DV, g);
 }

@@ -102,13 +102,39 @@ SGLC_API int sglc_xielu(const void* src, long long src_stride, int src_dtype, vo
 // columns from `n_weighted` on (an expert that every token uses, laid behind the routed ones) take 1.
 // `act` chooses the gate's function (silu, or the tanh form of GELU); `mult` is one more factor of
 // every result (a layer's residual multiplier, taken in 32-bit ahead of the rounding).
+// `pass` (rows of E, optional): the same launch also forms x[r][c] = w_pass[r] * h[r][c] (added to x
+// with `add`): the experts of a mixture that hand their input on as it is, summed straight into the
+// 32-bit rows that the down product adds to.
 enum { GA_SILU = 0, GA_GELU_TANH = 1 };
+struct PassRows {
+  const void* h; long long h_stride;      // in the activation precision (null: none)
+  const float* w;                         // [rows]
+  float* x; long long x_stride;
+  int E, add;
+};
+template <typename TI>
+__device__ __forceinline__ void pass_rows(const PassRows& p, int rows) {
+  if (!p.h) return;
+  const TI* h = static_cast<const TI*>(p.h);
+  const long long total = (long long)rows * p.E;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
+       i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / p.E;
+    const int c = (int)(i % p.E);
+    const float w = p.w[r];
+    float* xp = p.x + r * p.x_stride + c;
+    if (!p.add) *xp = w * to_f32(h[r * p.h_stride + c]);
+    else if (w != 0.0f) *xp = fmaf(w, to_f32(h[r * p.h_stride + c]), *xp);
+  }
+}
 template <typename TI, typename TO>
 __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_stride, TO* __restrict__ dst,
                                  long long dst_stride, int rows, int F, const float* __restrict__ w,
-                                 long long w_stride, int per, int act, float mult, int n_weighted) {
+                                 long long w_stride, int per, int act, float mult, int n_weighted,
+                                 const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
+  pass_rows<TO>(pass, rows);
   const long long total = (long long)rows * F;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
        i += (long long)gridDim.x * blockDim.x) {
@@ -129,9 +155,10 @@ __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_strid
 __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, long long src_stride,
                                       __nv_bfloat16* __restrict__ dst, long long dst_stride, int rows, int F,
                                       const float* __restrict__ w, long long w_stride, int per, int act, float mult,
-                                      int n_weighted) {
+                                      int n_weighted, const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
+  pass_rows<__nv_bfloat16>(pass, rows);
   const int F8 = F / 8;
   const long long total = (long long)rows * F8;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
@@ -160,9 +187,9 @@ __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, lon
 }
 
 // n_weighted: the first so many columns (a multiple of `per`) take weights, the rest take 1
-SGLC_API int sglc_gated_act_part(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
-                                 int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
-                                 int act, float mult, int n_weighted, cudaStream_t stream) {
+static int gated_act_run(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
+                         int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
+                         int act, float mult, int n_weighted, const PassRows& pass, cudaStream_t stream) {
   if (rows <= 0 || F <= 0) return SGLC_OK;
   if (act != GA_SILU && act != GA_GELU_TANH) return SGLC_ERR_ARGUMENT;
   if (w && (per <= 0 || n_weighted < 0 || n_weighted > F || n_weighted % per != 0)) return SGLC_ERR_ARGUMENT;
@@ -175,16 +202,36 @@ SGLC_API int sglc_gated_act_part(const void* src, long long src_stride, int src_
     if (b8 > 148 * 16) b8 = 148 * 16;
     return sglc_launch(gated_act_vec8_kernel, dim3(b8), dim3(256), 0, stream, 1, true, (const __nv_bfloat16*)src,
                        src_stride, (__nv_bfloat16*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult,
-                       n_weighted);
+                       n_weighted, pass);
   }
 #define LAUNCH(TI, TO)                                                                                  \
   return sglc_launch(gated_act_kernel<TI, TO>, dim3(blocks), dim3(256), 0, stream, 1, true, (const TI*)src, \
-                     src_stride, (TO*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult, n_weighted)
+                     src_stride, (TO*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult, n_weighted, pass)
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_F32) LAUNCH(float, float);
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_BF16) LAUNCH(float, __nv_bfloat16);
   if (src_dtype == SGLC_BF16 && dst_dtype == SGLC_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
 #undef LAUNCH
   return SGLC_ERR_ARGUMENT;
+}
+
+SGLC_API int sglc_gated_act_part(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
+                                 int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
+                                 int act, float mult, int n_weighted, cudaStream_t stream) {
+  PassRows none = {};
+  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per, act, mult,
+                       n_weighted, none, stream);
+}
+
+// With rows handed on: x[r][c] (+)= w_pass[r] * h[r][c], c < E; h in dst's precision, x 32-bit.
+SGLC_API int sglc_gated_act_pass(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
+                                 int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
+                                 int act, float mult, int n_weighted, const void* h, long long h_stride,
+                                 const float* w_pass, float* x, long long x_stride, int E, int add,
+                                 cudaStream_t stream) {
+  if (!h || !w_pass || !x || E <= 0) return SGLC_ERR_ARGUMENT;
+  PassRows pass = {h, h_stride, w_pass, x, x_stride, E, add};
+  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per, act, mult,
+                       n_weighted, pass, stream);
 }
 
 SGLC_API int sglc_gated_act_ext(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,

@@ -1,5 +1,5 @@
 // Token embedding gather with an optional additive position table:
-//   x[t,:] = wte[tok[t],:] (+ wpe[pos[t],:])      (reference src/gpt2.c:211-216,
+//   x[t,:] = wte[tok[t],:] * scale (+ wpe[pos[t],:])      (scale is 1 unless a model asks; reference src/gpt2.c:211-216,
 //   GPU twin k_embed_pos src/cuda_backend.cu:477-483).
 // Tables are float or bfloat16; the sum is formed and stored in 32-bit.
 #include "common.cuh"
@@ -9,7 +9,7 @@ SGLC_DEFINE_ERROR_STRING()
 template <typename TW>
 __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
                              const TW* __restrict__ wte, const TW* __restrict__ wpe,
-                             float* __restrict__ out, int T, int E, int V, int P,
+                             float* __restrict__ out, int T, int E, int V, int P, float scale,
                              int* __restrict__ err) {
   int t = blockIdx.x;
   if (t >= T) return;
@@ -32,28 +32,34 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
   const TW* b = wpe ? wpe + (size_t)pos * E : nullptr;
   float* o = out + (size_t)t * E;
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
-    float v = to_f32(a[e]);
+    float v = to_f32(a[e]) * scale;
     if (b) v += to_f32(b[e]);
     o[e] = v;
   }
 }
 
 // err: one int on the device, set to 1 if a token or position is out of range (may be null).
-SGLC_API int sglc_embed(const int* tokens, const int* positions, const void* wte, const void* wpe,
-                        float* out, int T, int E, int V, int P, int table_dtype, int* err,
-                        cudaStream_t stream) {
+SGLC_API int sglc_embed_scaled(const int* tokens, const int* positions, const void* wte, const void* wpe,
+                               float* out, int T, int E, int V, int P, int table_dtype, float scale, int* err,
+                               cudaStream_t stream) {
   if (T <= 0) return SGLC_OK;
   int threads = E >= 1024 ? 256 : (E >= 256 ? 128 : 64);
   if (table_dtype == SGLC_F32)
     return sglc_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, stream, 1, true, tokens,
-                       positions, (const float*)wte, (const float*)wpe, out, T, E, V, P, err);
+                       positions, (const float*)wte, (const float*)wpe, out, T, E, V, P, scale, err);
   else if (table_dtype == SGLC_BF16)
     return sglc_launch(embed_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, 1, true,
                        tokens, positions, (const __nv_bfloat16*)wte, (const __nv_bfloat16*)wpe, out, T,
-                       E, V, P, err);
+                       E, V, P, scale, err);
   else
     return SGLC_ERR_ARGUMENT;
   return sglc_launch_status();
+}
+
+SGLC_API int sglc_embed(const int* tokens, const int* positions, const void* wte, const void* wpe,
+                        float* out, int T, int E, int V, int P, int table_dtype, int* err,
+                        cudaStream_t stream) {
+  return sglc_embed_scaled(tokens, positions, wte, wpe, out, T, E, V, P, table_dtype, 1.0f, err, stream);
 }
 
 // x[t,:] += table[pos[t],:]  — a position table added after the gather, for

@@ -337,3 +337,147 @@ SGLC_API int sglc_norm_rows(const void* src, long long src_stride, int src_dtype
   return sglc_norm_rows_grouped(src, src_stride, src_dtype, src_rows, gain, bias, dst, dst_stride, dst_dtype, dst_rows,
                                 dst_row_limit, n_rows, E, eps, form, add, 1, err, stream);
 }
+
+// Two RMS norms of the same rows (parallel sublayers with a norm each) and, on the first one's
+// result, a token shift, in one launch, a block a token:
+//   h_t = x_t / sqrt(mean(x_t^2) + eps) * g1;   y1_t = h_t + (h_(t-1) - h_t) * mu;   y2_t likewise with g2
+// h_(t-1) is the token before of the same request, before its own shift; zero ahead of the first
+// token, and `prev[slot]` (kept in 32-bit) ahead of a portion's first.  The block of a portion's
+// FIRST token is the only one that touches the slot: it reads what the portion before left and then
+// writes the h of the portion's last token, which it norms itself, so nothing waits for another block.
+// Without mu: y1 = h.  Without y2: one norm.
+template <typename TO, bool VEC>
+__global__ void norm_pair_shift_kernel(const float* __restrict__ x, const float* __restrict__ g1,
+                                       const float* __restrict__ g2, const float* __restrict__ mu, float eps,
+                                       float* __restrict__ prev, const int* __restrict__ token_req,
+                                       const int* __restrict__ q_start, const int* __restrict__ state_slots,
+                                       TO* __restrict__ y1, long long y1_stride, TO* __restrict__ y2,
+                                       long long y2_stride, int E, int n_slots, int* __restrict__ err) {
+  extern __shared__ __align__(16) float srow[];   // the token's row; with mu, then the other row
+  __shared__ float red[2][33];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  pdl_launch_dependents();
+  // (the step's own arrays: no kernel of the step writes them)
+  int first = 0, last = 0, slot = -1;
+  if (mu) {
+    const int r = token_req[t];
+    first = q_start[r];
+    last = q_start[r + 1] - 1;
+    slot = state_slots[r];
+  }
+  const bool head = mu && t == first;             // this block serves the slot
+  const int other = !mu ? -1 : head ? last : t - 1;
+  float* orow = srow + E;
+  const int n_it = VEC ? E / 4 : E;
+  pdl_wait();
+  const float* xr = x + (size_t)t * E;
+  const float* xo = x + (size_t)(other < 0 ? t : other) * E;
+  const bool two = mu && other != t;              // (a single token's own row serves as the last one)
+  float qa = 0.0f, qb = 0.0f;
+  for (int i = threadIdx.x; i < n_it; i += blockDim.x) {
+    if constexpr (VEC) {
+      const float4 v = reinterpret_cast<const float4*>(xr)[i];
+      reinterpret_cast<float4*>(srow)[i] = v;
+      qa = sq4(v, 0.0f, qa);
+      if (two) {
+        const float4 o = reinterpret_cast<const float4*>(xo)[i];
+        reinterpret_cast<float4*>(orow)[i] = o;
+        qb = sq4(o, 0.0f, qb);
+      }
+    } else {
+      const float v = xr[i];
+      srow[i] = v;
+      qa = fmaf(v, v, qa);
+      if (two) {
+        const float o = xo[i];
+        orow[i] = o;
+        qb = fmaf(o, o, qb);
+      }
+    }
+  }
+  // both sums at once; the order of additions depends on the width only
+  qa = warp_sum(qa);
+  qb = warp_sum(qb);
+  if (lane == 0) { red[0][warp] = qa; red[1][warp] = qb; }
+  __syncthreads();
+  qa = 0.0f; qb = 0.0f;
+  for (int w = 0; w < nw; w++) { qa += red[0][w]; qb += red[1][w]; }
+  const float ia = 1.0f / sqrtf(qa / (float)E + eps);
+  const float ib = two ? 1.0f / sqrtf(qb / (float)E + eps) : ia;
+  const float* brow = two ? orow : srow;
+  float* ps = nullptr;
+  if (head) {
+    if (!sglc_index_ok(slot, n_slots, err)) return;
+    ps = prev + (size_t)slot * E;
+  }
+  TO* o1 = y1 + (size_t)t * y1_stride;
+  TO* o2 = y2 ? y2 + (size_t)t * y2_stride : nullptr;
+  // (a thread reads and writes the same columns of the rows it staged, so nothing more is waited for)
+  for (int i = threadIdx.x; i < n_it; i += blockDim.x) {
+    if constexpr (VEC) {
+      const float4 v = reinterpret_cast<const float4*>(srow)[i];
+      float4 h = norm4(v, 0.0f, ia, g1, nullptr, i);
+      if (mu) {
+        const float4 hb = norm4(reinterpret_cast<const float4*>(brow)[i], 0.0f, ib, g1, nullptr, i);
+        float4 p = hb;
+        if (head) {
+          p = reinterpret_cast<float4*>(ps)[i];
+          reinterpret_cast<float4*>(ps)[i] = hb;
+        }
+        const float4 m = reinterpret_cast<const float4*>(mu)[i];
+        h = make_float4(fmaf(p.x - h.x, m.x, h.x), fmaf(p.y - h.y, m.y, h.y), fmaf(p.z - h.z, m.z, h.z),
+                        fmaf(p.w - h.w, m.w, h.w));
+      }
+      store4<TO>(o1 + 4 * i, h);
+      if (o2) store4<TO>(o2 + 4 * i, norm4(v, 0.0f, ia, g2, nullptr, i));
+    } else {
+      const float n = __fmul_rn(srow[i], ia);
+      float h = g1 ? __fmul_rn(n, g1[i]) : n;
+      if (mu) {
+        float hb = __fmul_rn(brow[i], ib);
+        if (g1) hb = __fmul_rn(hb, g1[i]);
+        float p = hb;
+        if (head) {
+          p = ps[i];
+          ps[i] = hb;
+        }
+        h = fmaf(p - h, mu[i], h);
+      }
+      o1[i] = from_f32<TO>(h);
+      if (o2) o2[i] = from_f32<TO>(g2 ? __fmul_rn(n, g2[i]) : n);
+    }
+  }
+}
+
+// x: float [T][E] contiguous; g1, g2, mu: float [E] (g2 with y2 only; mu may be null); prev: float
+// [n_slots][E] (with mu); y1, y2 (y2 may be null): [T][stride] of out_dtype.
+SGLC_API int sglc_norm_pair_shift(const float* x, const float* g1, const float* g2, const float* mu, float eps,
+                                  float* prev, const int* token_req, const int* q_start, const int* state_slots,
+                                  void* y1, long long y1_stride, void* y2, long long y2_stride, int out_dtype, int T,
+                                  int E, int n_slots, int* err, cudaStream_t stream) {
+  if (T <= 0) return SGLC_OK;
+  if (E <= 0 || !y1 || (mu && (!prev || !token_req || !q_start || !state_slots))) return SGLC_ERR_ARGUMENT;
+  if (out_dtype != SGLC_F32 && out_dtype != SGLC_BF16) return SGLC_ERR_ARGUMENT;
+  const size_t smem = (size_t)E * (mu ? 2 : 1) * sizeof(float);
+  if (smem > 200 * 1024) return SGLC_ERR_UNSUPPORTED;
+  const int threads = E >= 2048 ? 512 : (E >= 512 ? 256 : (E >= 128 ? 128 : (E >= 64 ? 64 : 32)));
+  const int oa = out_dtype == SGLC_F32 ? 15 : 7;
+  const bool vec = E % 4 == 0 && al16(x) && al16(g1) && al16(g2) && al16(mu) && al16(prev) && y1_stride % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(y1) & oa) == 0 &&
+                   (!y2 || (y2_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(y2) & oa) == 0));
+#define PAIR(TO, VEC)                                                                                            \
+  do {                                                                                                           \
+    if (smem > 48 * 1024)                                                                                        \
+      cudaFuncSetAttribute(norm_pair_shift_kernel<TO, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    return sglc_launch(norm_pair_shift_kernel<TO, VEC>, dim3(T), dim3(threads), smem, stream, 1, true, x, g1, g2, mu, \
+                       eps, prev, token_req, q_start, state_slots, (TO*)y1, y1_stride, (TO*)y2, y2_stride, E, n_slots, \
+                       err);                                                                                     \
+  } while (0)
+  if (out_dtype == SGLC_BF16) {
+    if (vec) PAIR(__nv_bfloat16, true);
+    PAIR(__nv_bfloat16, false);
+  }
+  if (vec) PAIR(float, true);
+  PAIR(float, false);
+#undef PAIR
+}

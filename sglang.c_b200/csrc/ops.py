@@ -151,8 +151,8 @@ def _i32(t, what):
 
 
 # ---------------------------------------------------------------------------
-def embed(tokens, table, out, positions=None, pos_table=None, err_flag=None, inv_freq=None):
-    """out[t,:] = table[tokens[t],:] (+ pos_table[positions[t],:]); out is float32 [T,E].
+def embed(tokens, table, out, positions=None, pos_table=None, err_flag=None, inv_freq=None, scale=1.0):
+    """out[t,:] = table[tokens[t],:] * scale (+ pos_table[positions[t],:]); out is float32 [T,E].
     With inv_freq (float64 [ceil(E/2)]) instead of a position table, the sinusoidal vector
     sin/cos(positions[t] * inv_freq[i]) at entries 2i / 2i+1 is added."""
     _need_cuda(tokens, table, out, positions, pos_table, inv_freq)
@@ -164,6 +164,8 @@ def embed(tokens, table, out, positions=None, pos_table=None, err_flag=None, inv
         raise KernelError(f"embed: table {tuple(table.shape)} does not match width {E}")
     if inv_freq is not None:
         _i32(positions, "positions")
+        if scale != 1.0:
+            raise KernelError("embed: no scaled rows with computed positions")
         if pos_table is not None or inv_freq.dtype != torch.float64 or inv_freq.numel() != (E + 1) // 2 \
                 or not inv_freq.is_contiguous():
             raise KernelError("embed: inverse wavelengths must be float64, one per pair of columns, and come "
@@ -180,8 +182,9 @@ def embed(tokens, table, out, positions=None, pos_table=None, err_flag=None, inv
             raise KernelError("embed: position table must have the token table's dtype and width")
         P = pos_table.shape[0]
     lib = build.load("embed")
-    code = lib.sglc_embed(_ptr(tokens), _ptr(positions), _ptr(table), _ptr(pos_table), _ptr(out),
-                          T, E, table.shape[0], P, _dt(table, "embed table"), _ptr(err_flag), _stream())
+    code = lib.sglc_embed_scaled(_ptr(tokens), _ptr(positions), _ptr(table), _ptr(pos_table), _ptr(out),
+                                 T, E, table.shape[0], P, _dt(table, "embed table"), ctypes.c_float(scale),
+                                 _ptr(err_flag), _stream())
     _check(lib, code, "embed")
 
 
@@ -259,6 +262,18 @@ def kv_write(k_src, v_src, cache, slots, n_kv_heads, head_dim):
                              H, D, page_size, n_pages, _dt(k_src, "kv source"), _dt(cache, "cache"),
                              _stream())
     _check(lib, code, "kv_write")
+
+
+def _gate_args(gate, T, n_heads, width, what):
+    """(pointer, row stride, 1 if per head) of an output gate: float32 rows of pre-activations, [T, n_heads]
+    or [T, n_heads * width]; None: no gate."""
+    if gate is None:
+        return None, ctypes.c_longlong(0), 0
+    _need_cuda(gate)
+    _f32_rows(gate, f"{what}: gate")
+    if gate.shape[0] < T or gate.shape[1] not in (n_heads, n_heads * width):
+        raise KernelError(f"{what}: a gate has one number per head, or one per entry of the heads' results")
+    return _ptr(gate), ctypes.c_longlong(gate.stride(0)), 1 if gate.shape[1] == n_heads else 0
 
 
 def attention_simt(q, cache, block_table, token_req, positions, out, n_heads, scale, window,
@@ -576,12 +591,14 @@ def attention_latent_decode_supported(q, cache, n_heads):
 
 
 def attention_latent_decode(q, cache, block_table, token_req, positions, out, n_heads, scale, window, max_keys,
-                            token_list=None, n_tokens=None, n_splits=None):
+                            token_list=None, n_tokens=None, n_splits=None, sinks=None, gate=None):
     """Attention of single decoded tokens over a cached latent [n_pages, 1, 1, page_size, D] (rows
     that are keys and values of every head): one block serves all heads of a token over a range
     of its keys, so a row comes from memory once.  token_req None: token t belongs to the step's
-    t-th request.  token_list (int32, its first n_tokens entries): the tokens to serve."""
-    _need_cuda(q, cache, block_table, token_req, positions, out, token_list)
+    t-th request.  token_list (int32, its first n_tokens entries): the tokens to serve.  sinks: float32
+    [n_heads], a score per head that joins the softmax's denominator; gate: float32 pre-activations
+    [all tokens, n_heads] or [.., n_heads * dim] whose sigmoid multiplies the heads' results."""
+    _need_cuda(q, cache, block_table, token_req, positions, out, token_list, sinks)
     for t, nm in ((block_table, "block_table"), (positions, "positions")):
         _i32(t, nm)
     T = q.shape[0]
@@ -591,6 +608,9 @@ def attention_latent_decode(q, cache, block_table, token_req, positions, out, n_
         _i32(token_list, "token_list")
         T = int(n_tokens)
     n_pages, one, Hkv, page_size, D = cache.shape
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
+        raise KernelError("attention_latent_decode: one float32 sink per head")
+    gp, gs, per_head = _gate_args(gate, q.shape[0], n_heads, D, "attention_latent_decode")
     if one != 1 or Hkv != 1 or not cache.is_contiguous() or cache.dtype != torch.bfloat16 \
             or q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attention_latent_decode: bfloat16 queries and output, cache [n_pages,1,1,page,dim]")
@@ -605,7 +625,7 @@ def attention_latent_decode(q, cache, block_table, token_req, positions, out, n_
                                             block_table.stride(0), _ptr(token_req), _ptr(positions), _ptr(token_list),
                                             _ptr(out), out.stride(0), T, n_heads, D, page_size, ctypes.c_float(scale),
                                             int(window or 0), splits, _ptr(ws), ctypes.c_longlong(ws.numel()), n_pages,
-                                            _ptr(err), _stream())
+                                            _ptr(err), _ptr(sinks), gp, gs, per_head, _stream())
     _check(lib, code, f"attention_latent_decode (dim {D}, up to {max_keys} keys)", n_kernels=2 if splits > 1 else 1)
 
 
@@ -617,12 +637,13 @@ def attention_prefill_tc_supported(q, cache, scale):
 
 
 def attention_prefill_tc(q, cache, block_table, q_start, kv_len, out, n_heads, scale, window,
-                         n_requests, max_q_len, skip_single=False, kv_shared=False, chunk=None, sinks=None):
+                         n_requests, max_q_len, skip_single=False, kv_shared=False, chunk=None, sinks=None, gate=None):
     """Causal attention of prompt portions on the tensor cores (tcgen05), bfloat16, head
     sizes 64 and 128.  q_start int32 [R+1], kv_len int32 [R] (lengths after this step).
     kv_shared: cache is [n_pages, 1, n_kv_heads, page_size, head_dim], rows that are keys and
     values at once.  chunk: a query sees only the keys of its own chunk of so many positions;
-    sinks: float32 [n_heads], a score per head that joins the softmax's denominator."""
+    sinks: float32 [n_heads], a score per head that joins the softmax's denominator; gate: float32
+    pre-activations [T, n_heads] or [T, n_heads * head_dim] whose sigmoid multiplies the heads' results."""
     _need_cuda(q, cache, block_table, q_start, kv_len, out, sinks)
     for t, nm in ((block_table, "block_table"), (q_start, "q_start"), (kv_len, "kv_len")):
         _i32(t, nm)
@@ -637,15 +658,15 @@ def attention_prefill_tc(q, cache, block_table, q_start, kv_len, out, n_heads, s
         raise KernelError(f"attention_prefill_tc: cache {tuple(cache.shape)} does not fit kv_shared={kv_shared}")
     lib = build.load("attention_prefill_tc")
     err = _tc_buffers(q.device)[2]
-    if chunk or sinks is not None:
-        if kv_shared or (sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads)):
-            raise KernelError("attention_prefill_tc: a chunk mask or sinks go with separate keys and values; "
-                              "one float32 sink per head")
+    if chunk or sinks is not None or gate is not None:
+        if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
+            raise KernelError("attention_prefill_tc: one float32 sink per head")
+        gp, gs, per_head = _gate_args(gate, q.shape[0], n_heads, D, "attention_prefill_tc")
         code = lib.sglc_attention_prefill_tc_ext(
             _ptr(q), q.stride(0), _ptr(cache), _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len),
             _ptr(out), out.stride(0), int(n_requests), int(max_q_len), n_heads, Hkv, D, page_size,
             ctypes.c_float(scale), int(window or 0), int(chunk or 0), _ptr(sinks), q.shape[0], n_pages,
-            1 if skip_single else 0, _ptr(err), _stream())
+            1 if skip_single else 0, _ptr(err), 1 if kv_shared else 0, gp, gs, per_head, _stream())
         _check(lib, code, f"attention_prefill_tc (head_dim {D}, chunk {chunk})")
         return
     fn = lib.sglc_attention_prefill_tc_shared if kv_shared else lib.sglc_attention_prefill_tc
@@ -748,6 +769,35 @@ def norm_add_tail(y, gain, eps, x, form="layer", mix=None, then=None):
                                   ctypes.c_longlong(out.stride(0) if out is not None else 0),
                                   _dt(out, "norm output") if out is not None else F32, n, E, _stream())
     _check(lib, code, f"norm_add_tail (width {E})")
+
+
+def norm_pair_shift(x, gain1, gain2, eps, y1, y2, shift=None, prev=None, token_req=None, q_start=None, state_slots=None):
+    """y1 = rms_norm(x) * gain1 and y2 = rms_norm(x) * gain2 in one launch (y2 None: the first alone);
+    with `shift` (float32 [E]) y1[t] is moved towards the row of the request's token before,
+    y1[t] += (h[t-1] - h[t]) * shift, h being the normed rows before that: prev float32 [n_slots, E]
+    holds every request's last one, read and replaced in place.  x float32 [T, E] contiguous."""
+    _need_cuda(x, gain1, gain2, y1, y2, shift, prev, token_req, q_start, state_slots)
+    T, E = y1.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.shape[1] != E or x.shape[0] < T or y1.stride(1) != 1 \
+            or (y2 is not None and (y2.dtype != y1.dtype or y2.shape != y1.shape or y2.stride(1) != 1)):
+        raise KernelError("norm_pair_shift: x contiguous float32 [T, E]; both results [T, E] of one dtype")
+    for g, nm in ((gain1, "gain"), (gain2, "gain"), (shift, "shift")):
+        if g is not None and (g.dtype != torch.float32 or g.numel() != E or not g.is_contiguous()):
+            raise KernelError(f"norm_pair_shift: a {nm} is a float32 vector of {E}")
+    n_slots = 0
+    if shift is not None:
+        for t, nm in ((token_req, "token_req"), (q_start, "q_start"), (state_slots, "state_slots")):
+            _i32(t, nm)
+        if prev is None or prev.dtype != torch.float32 or not prev.is_contiguous() or prev.shape[1:] != (E,):
+            raise KernelError(f"norm_pair_shift: prev is float32 [n_slots, {E}]")
+        n_slots = prev.shape[0]
+    lib = build.load("norm_rows")
+    code = lib.sglc_norm_pair_shift(
+        _ptr(x), _ptr(gain1), _ptr(gain2), _ptr(shift), ctypes.c_float(eps), _ptr(prev), _ptr(token_req), _ptr(q_start),
+        _ptr(state_slots), _ptr(y1), ctypes.c_longlong(y1.stride(0)), _ptr(y2),
+        ctypes.c_longlong(y2.stride(0) if y2 is not None else 0), _dt(y1, "norm_pair_shift"), T, E, n_slots,
+        _ptr(tc_error_flag(x.device)), _stream())
+    _check(lib, code, f"norm_pair_shift (width {E})")
 
 
 GATED_SCAN_CHUNK = 128      # a step whose longest portion exceeds this goes the gated scans' chunked way ...
@@ -1005,14 +1055,17 @@ QK_NORMS = {None: 0, False: 0, "none": 0, True: 1, "unit": 1, "head_gain": 2, "r
 
 
 def qk_prep(x, positions, freq, mult, dims, pairing, norm, eps, gain_q, gain_k, q_out, cache, slots, n_heads,
-            n_kv_heads, dim, v_dim, page_size, v_mult=1.0):
+            n_kv_heads, dim, v_dim, page_size, v_mult=1.0, conv=None):
     """The general input stage of a softmax attention (rotary.cu: qk_prep_kernel).  x: float32 rows
     [T, H*dim | G*dim | G*v_dim], or [T, H*dim] alone with n_kv_heads = 0 (a layer that reads keys and
     values another layer cached: cache and slots are then None).  norm: None; "unit" (after the
     turn, no gain); "head_gain" (before the turn, per head, gains float32 [dim] shared by the heads);
     "row_gain" (before the turn, one root mean square over all query heads and one over all key
     heads, gains float32 [H*dim] and [G*dim]).  pairing "halves" or "neighbours".  Queries go to q_out
-    [T, H*dim]; keys and values (times v_mult) into the cache's pages at slots."""
+    [T, H*dim]; keys and values (times v_mult) into the cache's pages at slots.
+    conv = (taps, tail, token_req, q_start, state_slots, n_requests): x's channels first pass a causal
+    convolution over time; taps float32 [K, C] (the last row is the current token's), tail float32
+    [n_slots, K-1, C], every request's last K-1 inputs, read and moved on in place."""
     _need_cuda(x, positions, freq, q_out, cache, slots, gain_q, gain_k)
     T = q_out.shape[0]
     G = int(n_kv_heads)
@@ -1036,6 +1089,31 @@ def qk_prep(x, positions, freq, mult, dims, pairing, norm, eps, gain_q, gain_k, 
         for g, n, nm in ((gain_q, want[0], "queries"), (gain_k, want[1], "keys")):
             if n and (g is None or g.dtype != torch.float32 or g.numel() != n or not g.is_contiguous()):
                 raise KernelError(f"qk_prep: the gain of the {nm} is a float32 vector of {n}")
+    if conv is not None:
+        taps, tail, token_req, q_start, state_slots, R = conv
+        _need_cuda(taps, tail, token_req, q_start, state_slots)
+        K, C = taps.shape
+        for t, nm in ((token_req, "token_req"), (q_start, "q_start"), (state_slots, "state_slots")):
+            _i32(t, nm)
+        if C != x.shape[1] or taps.dtype != torch.float32 or not taps.is_contiguous() or tail.dtype != torch.float32 \
+                or not tail.is_contiguous() or tuple(tail.shape[1:]) != (K - 1, C):
+            raise KernelError(f"qk_prep: taps float32 [K, {x.shape[1]}], tail float32 [n_slots, K-1, {x.shape[1]}]")
+        own = T == int(R)
+        lib, tlib = build.load("rotary"), build.load("short_conv")
+        flag = _ptr(tc_error_flag(x.device))
+        code = lib.sglc_qk_prep_conv(
+            _ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(positions), _ptr(freq if dims else None), ctypes.c_float(mult),
+            int(dims), ROTARY_PAIRINGS[pairing], mode, ctypes.c_float(eps or 0.0), _ptr(gain_q),
+            _ptr(gain_k if G else None), ctypes.c_float(v_mult), _ptr(q_out), ctypes.c_longlong(q_out.stride(0)),
+            _ptr(cache if G else None), _ptr(slots if G else None), T, int(n_heads), G, int(dim), int(v_dim),
+            int(page_size), n_pages, _dt(q_out, "queries"), flag, _ptr(taps), _ptr(tail), _ptr(token_req), _ptr(q_start),
+            _ptr(state_slots), K, tail.shape[0], 1 if own else 0, _stream())
+        _check(lib, code, f"qk_prep (head {dim}, {K} taps)")
+        if K > 1 and not own:
+            code = tlib.sglc_short_conv_tail(_ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(tail), _ptr(q_start),
+                                             _ptr(state_slots), int(R), C, K, tail.shape[0], flag, _stream())
+            _check(tlib, code, "short_conv_tail")
+        return
     lib = build.load("rotary")
     code = lib.sglc_qk_prep(_ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(positions), _ptr(freq if dims else None),
                             ctypes.c_float(mult), int(dims), ROTARY_PAIRINGS[pairing], mode, ctypes.c_float(eps or 0.0),
@@ -1098,13 +1176,17 @@ def attention_ext_splits(max_keys, window=None, chunk=None):
 
 
 def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_kv_heads, dim, v_dim, page_size,
-                  scale, window, chunk, sinks, max_keys, max_q_len=None, splits=1, workspace=None):
+                  scale, window, chunk, sinks, max_keys, max_q_len=None, splits=1, workspace=None, kv_shared=False,
+                  gate=None):
     """attention_simt's extended form: values of size v_dim beside keys of size dim (cache
     [n_pages, G*page_size*(dim+v_dim)]: a page's keys, then its values), an optional chunk mask
     (a query sees the keys of its own chunk of `chunk` positions) and an optional sink per head
     (float32 [H]) in the softmax's denominator.  q [T, H*dim]; out [T, H*v_dim].
     splits > 1 (a step of single tokens only): every token's keys are dealt to so many blocks, whose
-    shares a second launch merges; workspace: float32, T * H * splits * (v_dim + 2) entries."""
+    shares a second launch merges; workspace: float32, T * H * splits * (v_dim + 2) entries.
+    kv_shared: the cache keeps one row of `dim` entries per position and head, a key whose first v_dim
+    entries are its value.  splits None: chosen here, with the library's own scratch.  gate: float32 pre-activations [T, H] or [T, H*v_dim] whose sigmoid
+    multiplies the heads' results."""
     _need_cuda(q, cache, block_table, token_req, positions, out, sinks, workspace)
     for t, nm in ((block_table, "block_table"), (token_req, "token_req"), (positions, "positions")):
         _i32(t, nm)
@@ -1113,11 +1195,18 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
     if q.shape[1] != n_heads * dim or out.shape[1] != n_heads * v_dim or q.stride(1) != 1 or out.stride(1) != 1 \
             or q.dtype != out.dtype or q.dtype != cache.dtype or not cache.is_contiguous():
         raise KernelError("attention_ext: q [T, H*dim], out [T, H*v_dim] and the cache have one dtype")
-    if cache.numel() != n_pages * n_kv_heads * page_size * (dim + v_dim):
+    if cache.numel() != n_pages * n_kv_heads * page_size * (dim if kv_shared else dim + v_dim) or (kv_shared and v_dim > dim):
         raise KernelError(f"attention_ext: cache {tuple(cache.shape)} does not fit {n_kv_heads} heads of {dim}+{v_dim}")
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads):
         raise KernelError("attention_ext: one float32 sink per head")
+    gp, gs, per_head = _gate_args(gate, T, n_heads, v_dim, "attention_ext")
     lib = build.load("attention_simt")
+    if splits is None:
+        splits = 1
+        if max_q_len == 1:
+            workspace = _tc_buffers(q.device)[0]
+            splits = min(attention_ext_splits(max_keys, window, chunk), workspace.numel() // (T * n_heads * (v_dim + 2)))
+            splits = max(splits, 1)
     if splits > 1:
         if (max_q_len or 2) > 1 or workspace is None or workspace.dtype != torch.float32 \
                 or workspace.numel() < T * n_heads * splits * (v_dim + 2) or not workspace.is_contiguous():
@@ -1127,8 +1216,8 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
             _ptr(q), q.stride(0), _ptr(cache), _ptr(block_table), block_table.stride(0), _ptr(token_req),
             _ptr(positions), _ptr(out), out.stride(0), T, int(n_heads), int(n_kv_heads), int(dim), int(v_dim),
             int(page_size), ctypes.c_float(scale), int(window or 0), int(chunk or 0), _ptr(sinks), int(max_keys),
-            _dt(q, "attention q"), _dt(cache, "cache"), n_pages, _ptr(tc_error_flag(q.device)), int(splits),
-            _ptr(workspace), _stream())
+            _dt(q, "attention q"), _dt(cache, "cache"), n_pages, _ptr(tc_error_flag(q.device)), 1 if kv_shared else 0,
+            gp, gs, per_head, int(splits), _ptr(workspace), _stream())
         _check(lib, code, f"attention_ext (head {dim}/{v_dim}, up to {max_keys} keys, {splits} shares)", n_kernels=2)
         return
     code = lib.sglc_attention_simt_ext(_ptr(q), q.stride(0), _ptr(cache), _ptr(block_table), block_table.stride(0),
@@ -1136,18 +1225,21 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
                                        int(n_kv_heads), int(dim), int(v_dim), int(page_size), ctypes.c_float(scale),
                                        int(window or 0), int(chunk or 0), _ptr(sinks), int(max_keys),
                                        _dt(q, "attention q"), _dt(cache, "cache"), n_pages,
-                                       _ptr(tc_error_flag(q.device)), int(max_q_len) if max_q_len else 2, _stream())
+                                       _ptr(tc_error_flag(q.device)), int(max_q_len) if max_q_len else 2,
+                                       1 if kv_shared else 0, gp, gs, per_head, _stream())
     _check(lib, code, f"attention_ext (head {dim}/{v_dim}, up to {max_keys} keys)")
 
 
 GATE_ACTS = {"silu": 0, "gelu_tanh": 1}
 
 
-def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=None):
+def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=None, handed_on=None):
     """dst[r, j] = act(src[r, j]) * src[r, F + j] (* weights[r, j // per]) * mult; src [rows, 2F] holds
     the gate columns, then the up columns; weights: float32 [rows, F // per] or None; act "silu" or
     "gelu_tanh"; mult: one more factor of every result, taken in 32-bit.  n_weighted: only the
-    first so many columns (a multiple of per) take weights, [rows, n_weighted // per]; the rest take 1."""
+    first so many columns (a multiple of per) take weights, [rows, n_weighted // per]; the rest take 1.
+    handed_on = (h, w, x, add): the same launch forms x[r, :] = w[r] * h[r, :] (added to x if `add`);
+    h [rows, E] in dst's dtype, w float32 [rows], x float32 [rows, E]."""
     _need_cuda(src, dst, weights)
     rows, F = dst.shape
     if src.shape[1] != 2 * F or src.shape[0] < rows or src.stride(1) != 1 or dst.stride(1) != 1:
@@ -1160,6 +1252,21 @@ def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=No
     else:
         nw = F
     lib = build.load("elementwise")
+    if handed_on is not None:
+        h, w, x, add = handed_on
+        _need_cuda(h, w, x)
+        _f32_rows(x, "gated_act: handed-on rows")
+        if h.dtype != dst.dtype or h.stride(1) != 1 or h.shape != x.shape or h.shape[0] != rows \
+                or w.dtype != torch.float32 or w.numel() < rows or not w.is_contiguous():
+            raise KernelError("gated_act: handed-on rows h [rows, E] in dst's dtype, w float32 [rows], x float32 [rows, E]")
+        code = lib.sglc_gated_act_pass(
+            _ptr(src), ctypes.c_longlong(src.stride(0)), _dt(src, "gated_act source"), _ptr(dst),
+            ctypes.c_longlong(dst.stride(0)), _dt(dst, "gated_act destination"), rows, F, _ptr(weights),
+            ctypes.c_longlong(weights.stride(0) if weights is not None else 0), int(per), GATE_ACTS[act],
+            ctypes.c_float(mult), nw, _ptr(h), ctypes.c_longlong(h.stride(0)), _ptr(w), _ptr(x),
+            ctypes.c_longlong(x.stride(0)), h.shape[1], 1 if add else 0, _stream())
+        _check(lib, code, "gated_act")
+        return
     code = lib.sglc_gated_act_part(_ptr(src), ctypes.c_longlong(src.stride(0)), _dt(src, "gated_act source"), _ptr(dst),
                                    ctypes.c_longlong(dst.stride(0)), _dt(dst, "gated_act destination"), rows, F,
                                    _ptr(weights), ctypes.c_longlong(weights.stride(0) if weights is not None else 0),
@@ -1171,13 +1278,15 @@ ROUTER_MAX_EXPERTS = 256
 
 
 def router(logits, correction, dense, ids, weights, top, n_groups=1, keep=1, renorm=False, weight_scale=1.0,
-           score="sigmoid", renorm_eps=0.0):
+           score="sigmoid", renorm_eps=0.0, group_score="top2_sum", n_pass=0, handed_on=None):
     """Routing by sigmoid scores (or, score "softmax", a softmax over all experts) with a choice
     correction and group limits; renorm: the chosen scores divided by their sum + renorm_eps; then
     times weight_scale (see router.cu).  logits: float32
     [T, E]; correction: float32 [E] or None; dense: float32 [T, E] (weights, zero where not
-    chosen); ids int32 [T, top]; weights float32 [T, top]."""
-    _need_cuda(logits, correction, dense, ids, weights)
+    chosen); ids int32 [T, top]; weights float32 [T, top].  group_score: "top2_sum", or "max" (a group
+    counts as its best expert).  handed_on (float32 [T]): takes the sum of a token's weights for the
+    last n_pass experts."""
+    _need_cuda(logits, correction, dense, ids, weights, handed_on)
     T, E = dense.shape
     _f32_rows(logits, "router: logits", E)
     _f32_rows(dense, "router: dense", E)
@@ -1187,10 +1296,14 @@ def router(logits, correction, dense, ids, weights, top, n_groups=1, keep=1, ren
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
         raise KernelError("router: one float32 correction per expert")
     lib = build.load("router")
-    code = lib.sglc_router_ext(_ptr(logits), ctypes.c_longlong(logits.stride(0)), _ptr(correction), _ptr(dense),
+    if handed_on is not None and (handed_on.dtype != torch.float32 or handed_on.numel() < T
+                                  or not handed_on.is_contiguous()):
+        raise KernelError("router: handed_on is float32 [T]")
+    code = lib.sglc_router_pass(_ptr(logits), ctypes.c_longlong(logits.stride(0)), _ptr(correction), _ptr(dense),
                                ctypes.c_longlong(dense.stride(0)), _ptr(ids), _ptr(weights), T, E, int(top),
                                int(n_groups), int(keep), 1 if renorm else 0, ctypes.c_float(weight_scale),
-                               {"sigmoid": 0, "softmax": 1}[score], ctypes.c_float(renorm_eps), _stream())
+                               {"sigmoid": 0, "softmax": 1}[score], ctypes.c_float(renorm_eps),
+                               {"top2_sum": 0, "max": 1}[group_score], int(n_pass), _ptr(handed_on), _stream())
     _check(lib, code, f"router ({E} experts, {top} chosen)")
 
 

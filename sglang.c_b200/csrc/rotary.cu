@@ -188,17 +188,33 @@ SGLC_API int sglc_latent_rope(const float* qx, long long qx_stride, const float*
 // (G x page_size x D keys, then G x page_size x V values) at slots[t]; values are multiplied by
 // v_mult on the way (a mixer whose result is a fixed multiple of the attention's folds it here:
 // the attention is linear in its values).  eps lies inside every root.
+// CONV: every channel of x first passes a causal convolution over time,
+//   u_t[ch] = sum_{j < K} taps[j][ch] * x_{t-(K-1)+j}[ch]     (no activation),
+// whose inputs ahead of a portion's first token are the request's tail[slot][m][ch] (m = 0 the
+// oldest of its last K-1 inputs; zero at a request's start).  In a step of single tokens (own_tail)
+// the thread that reads a channel's tail moves it on; otherwise a launch behind this one does
+// (short_conv.cu: short_conv_tail_kernel), when nobody reads a tail any more.
 constexpr int QK_WARPS = 8;      // (a token's head rows are dealt to the warps: eight keep the rounds few)
 
-template <typename TA>
+struct QkConv {
+  const float* taps;              // [K][C], C = H*D + G*(D+V)
+  float* tail;                    // [n_slots][K-1][C]
+  const int* token_req;           // [T]
+  const int* q_start;             // [R+1]
+  const int* state_slots;         // [R]
+  int K, n_slots, own_tail;
+};
+
+template <typename TA, bool CONV>
 __global__ void __launch_bounds__(QK_WARPS * 32)
 qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __restrict__ positions,
                const double* __restrict__ freq, float mult, int dims, int pairing, int norm_mode, float eps,
                const float* __restrict__ gain_q, const float* __restrict__ gain_k, float v_mult,
                TA* __restrict__ q_out, long long q_stride, TA* __restrict__ cache, const int* __restrict__ slots,
-               int T, int H, int G, int D, int V, int page_size, int n_pages, int* err) {
+               int T, int H, int G, int D, int V, int page_size, int n_pages, int* err, const QkConv cv) {
   __shared__ float buf[QK_WARPS][ROT_MAX_DIM];
   __shared__ float red[2][QK_WARPS];
+  extern __shared__ __align__(16) float conv_row[];      // CONV: the token's convolved channels
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
@@ -208,6 +224,27 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
   const bool page_ok = G > 0 && slot >= 0 && sglc_index_ok(page, n_pages, err);
   const size_t page_elems = (size_t)G * page_size * (D + V);
   const float* xr = x + (size_t)t * x_stride;
+  if constexpr (CONV) {
+    const int C = H * D + G * (D + V), K = cv.K;
+    const int r = cv.token_req[t], i = t - cv.q_start[r], slot_r = cv.state_slots[r];
+    if (!sglc_index_ok(slot_r, cv.n_slots, err)) return;
+    float* tail = cv.tail + (size_t)slot_r * (K - 1) * C;
+    for (int ch = threadIdx.x; ch < C; ch += QK_WARPS * 32) {
+      float acc = 0.0f;
+      for (int j = 0; j < K; j++) {
+        const int back = K - 1 - j;            // the input so many tokens ago
+        const float v = back <= i ? xr[ch - (long long)back * x_stride] : tail[(size_t)(K - 1 + i - back) * C + ch];
+        acc = fmaf(cv.taps[(size_t)j * C + ch], v, acc);
+      }
+      conv_row[ch] = acc;
+      if (cv.own_tail && K > 1) {              // (ascending: an entry is read before its place is written)
+        for (int m = 0; m + 1 < K - 1; m++) tail[(size_t)m * C + ch] = tail[(size_t)(m + 1) * C + ch];
+        tail[(size_t)(K - 2) * C + ch] = xr[ch];
+      }
+    }
+    __syncthreads();
+    xr = conv_row;
+  }
   const int half = dims / 2;
   float inv_all[2] = {1.0f, 1.0f};
   if (norm_mode == 3) {
@@ -286,10 +323,11 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
 
 // x: float [T][H*D (+ G*D + G*V)]; G = 0: queries only (cache and slots unused); gain_q, gain_k:
 // float, [D] each (norm_mode 2) or [H*D] and [G*D] (norm_mode 3), else unused.
-SGLC_API int sglc_qk_prep(const float* x, long long x_stride, const int* positions, const double* freq, float mult,
-                          int dims, int pairing, int norm_mode, float eps, const float* gain_q, const float* gain_k,
-                          float v_mult, void* q_out, long long q_stride, void* cache, const int* slots, int T, int H,
-                          int G, int D, int V, int page_size, int n_pages, int dtype, int* err, cudaStream_t stream) {
+static int qk_prep_run(const float* x, long long x_stride, const int* positions, const double* freq, float mult,
+                       int dims, int pairing, int norm_mode, float eps, const float* gain_q, const float* gain_k,
+                       float v_mult, void* q_out, long long q_stride, void* cache, const int* slots, int T, int H,
+                       int G, int D, int V, int page_size, int n_pages, int dtype, int* err, cudaStream_t stream,
+                       const QkConv* conv) {
   if (T <= 0) return SGLC_OK;
   if (H <= 0 || G < 0 || D <= 0 || V <= 0 || dims < 0 || dims > D || dims % 2 != 0 || page_size <= 0 ||
       norm_mode < 0 || norm_mode > 3 || (pairing != 0 && pairing != 1))
@@ -298,14 +336,54 @@ SGLC_API int sglc_qk_prep(const float* x, long long x_stride, const int* positio
   if (G > 0 && (!cache || !slots)) return SGLC_ERR_ARGUMENT;
   if (dims > 0 && !freq) return SGLC_ERR_ARGUMENT;
   if (D > ROT_MAX_DIM) return SGLC_ERR_UNSUPPORTED;
-  if (dtype == SGLC_F32)
-    return sglc_launch(qk_prep_kernel<float>, dim3(T), dim3(QK_WARPS * 32), 0, stream, 1, true, x, x_stride, positions,
-                       freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, (float*)q_out, q_stride,
-                       (float*)cache, slots, T, H, G, D, V, page_size, n_pages, err);
-  if (dtype == SGLC_BF16)
-    return sglc_launch(qk_prep_kernel<__nv_bfloat16>, dim3(T), dim3(QK_WARPS * 32), 0, stream, 1, true, x, x_stride,
-                       positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult,
-                       (__nv_bfloat16*)q_out, q_stride, (__nv_bfloat16*)cache, slots, T, H, G, D, V, page_size, n_pages,
-                       err);
+  QkConv cv = {};
+  size_t smem = 0;
+  if (conv) {
+    cv = *conv;
+    if (cv.K < 1 || !cv.taps || !cv.token_req || !cv.q_start || !cv.state_slots || (cv.K > 1 && !cv.tail))
+      return SGLC_ERR_ARGUMENT;
+    smem = ((size_t)H * D + (size_t)G * (D + V)) * sizeof(float);
+    if (smem > 200 * 1024) return SGLC_ERR_UNSUPPORTED;
+  }
+#define PREP(TA, CV)                                                                                               \
+  do {                                                                                                             \
+    if (smem > 24 * 1024)                                                                                          \
+      cudaFuncSetAttribute(qk_prep_kernel<TA, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
+    return sglc_launch(qk_prep_kernel<TA, CV>, dim3(T), dim3(QK_WARPS * 32), smem, stream, 1, true, x, x_stride,   \
+                       positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, (TA*)q_out,   \
+                       q_stride, (TA*)cache, slots, T, H, G, D, V, page_size, n_pages, err, cv);                   \
+  } while (0)
+  if (dtype == SGLC_F32) {
+    if (conv) PREP(float, true);
+    PREP(float, false);
+  }
+  if (dtype == SGLC_BF16) {
+    if (conv) PREP(__nv_bfloat16, true);
+    PREP(__nv_bfloat16, false);
+  }
+#undef PREP
   return SGLC_ERR_ARGUMENT;
+}
+
+SGLC_API int sglc_qk_prep(const float* x, long long x_stride, const int* positions, const double* freq, float mult,
+                          int dims, int pairing, int norm_mode, float eps, const float* gain_q, const float* gain_k,
+                          float v_mult, void* q_out, long long q_stride, void* cache, const int* slots, int T, int H,
+                          int G, int D, int V, int page_size, int n_pages, int dtype, int* err, cudaStream_t stream) {
+  return qk_prep_run(x, x_stride, positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, q_out,
+                     q_stride, cache, slots, T, H, G, D, V, page_size, n_pages, dtype, err, stream, nullptr);
+}
+
+// The same behind a causal convolution of K taps over the channels of x (which is [q | k | v], or q
+// alone with G = 0): taps [K][C], tail [n_slots][K-1][C].  own_tail: every request of the step brings
+// one token, and the kernel moves the tails on itself.
+SGLC_API int sglc_qk_prep_conv(const float* x, long long x_stride, const int* positions, const double* freq, float mult,
+                               int dims, int pairing, int norm_mode, float eps, const float* gain_q,
+                               const float* gain_k, float v_mult, void* q_out, long long q_stride, void* cache,
+                               const int* slots, int T, int H, int G, int D, int V, int page_size, int n_pages,
+                               int dtype, int* err, const float* taps, float* tail, const int* token_req,
+                               const int* q_start, const int* state_slots, int K, int n_slots, int own_tail,
+                               cudaStream_t stream) {
+  QkConv cv = {taps, tail, token_req, q_start, state_slots, K, n_slots, own_tail};
+  return qk_prep_run(x, x_stride, positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, q_out,
+                     q_stride, cache, slots, T, H, G, D, V, page_size, n_pages, dtype, err, stream, &cv);
 }

@@ -6,6 +6,9 @@
 //   a chosen expert's weight is its s (times `weight_scale`; with `renorm` the chosen weights
 //   are first divided by their sum plus `renorm_eps`).
 // `score_fn` 1: s = softmax(z) over all experts instead of the sigmoid.
+// `group_fn` 1: a group's score is its largest choice score instead of the sum of its two largest.
+// Of the E experts the last `n_pass` may be ones that hand their input on as it is: `pass` [T] (if
+// given) takes the sum of the token's weights for them.
 // Ties go to the lower index.  Results: dense [T][E] weights (zero where not chosen), and the
 // chosen ids and weights [T][top] in order of choice.  A thread a token; all 32-bit.
 #include "common.cuh"
@@ -19,7 +22,7 @@ __global__ void __launch_bounds__(64)
 router_kernel(const float* __restrict__ z, long long z_stride, const float* __restrict__ correction,
               float* __restrict__ dense, long long dense_stride, int* __restrict__ ids, float* __restrict__ wts,
               int T, int E, int top, int n_groups, int keep, int renorm, float weight_scale, int score_fn,
-              float renorm_eps) {
+              float renorm_eps, int group_fn, int n_pass, float* __restrict__ pass) {
   pdl_launch_dependents();
   const int t = blockIdx.x * 64 + threadIdx.x;
   pdl_wait();
@@ -47,7 +50,7 @@ router_kernel(const float* __restrict__ z, long long z_stride, const float* __re
         if (v > a) { b = a; a = v; }
         else if (v > b) b = v;
       }
-      gscore[g] = per > 1 ? a + b : a;
+      gscore[g] = per > 1 && group_fn == 0 ? a + b : a;
     }
     // the groups that stay: the `keep` best; the others' experts leave the choice
     unsigned long long kept = 0ull;
@@ -73,25 +76,38 @@ router_kernel(const float* __restrict__ z, long long z_stride, const float* __re
     c[best] = NAN;                             // taken
   }
   const float f = (renorm ? 1.0f / (sum + renorm_eps) : 1.0f) * weight_scale;
+  float handed_on = 0.0f;
   for (int n = 0; n < top; n++) {
     const float w = wts[(size_t)t * top + n] * f;
     wts[(size_t)t * top + n] = w;
     dense[(size_t)t * dense_stride + ids[(size_t)t * top + n]] = w;
+    if (ids[(size_t)t * top + n] >= E - n_pass) handed_on += w;
   }
+  if (pass) pass[t] = handed_on;
+}
+
+SGLC_API int sglc_router_pass(const float* z, long long z_stride, const float* correction, float* dense,
+                              long long dense_stride, int* ids, float* wts, int T, int E, int top, int n_groups,
+                              int keep, int renorm, float weight_scale, int score_fn, float renorm_eps,
+                              int group_fn, int n_pass, float* pass, cudaStream_t stream) {
+  if (T <= 0) return SGLC_OK;
+  if (E <= 0 || top <= 0 || top > E || n_groups < 1 || E % n_groups != 0 || keep < 1 || keep > n_groups)
+    return SGLC_ERR_ARGUMENT;
+  if (E > ROUTER_MAX_EXPERTS || n_groups > ROUTER_MAX_GROUPS) return SGLC_ERR_UNSUPPORTED;
+  if (n_groups > 1 && keep < n_groups && top > keep * (E / n_groups)) return SGLC_ERR_ARGUMENT;
+  if ((score_fn != 0 && score_fn != 1) || (group_fn != 0 && group_fn != 1) || n_pass < 0 || n_pass > E)
+    return SGLC_ERR_ARGUMENT;
+  return sglc_launch(router_kernel, dim3((T + 63) / 64), dim3(64), 0, stream, 1, true, z, z_stride, correction, dense,
+                     dense_stride, ids, wts, T, E, top, n_groups, keep, renorm, weight_scale, score_fn, renorm_eps,
+                     group_fn, n_pass, pass);
 }
 
 SGLC_API int sglc_router_ext(const float* z, long long z_stride, const float* correction, float* dense,
                              long long dense_stride, int* ids, float* wts, int T, int E, int top, int n_groups,
                              int keep, int renorm, float weight_scale, int score_fn, float renorm_eps,
                              cudaStream_t stream) {
-  if (T <= 0) return SGLC_OK;
-  if (E <= 0 || top <= 0 || top > E || n_groups < 1 || E % n_groups != 0 || keep < 1 || keep > n_groups)
-    return SGLC_ERR_ARGUMENT;
-  if (E > ROUTER_MAX_EXPERTS || n_groups > ROUTER_MAX_GROUPS) return SGLC_ERR_UNSUPPORTED;
-  if (n_groups > 1 && keep < n_groups && top > keep * (E / n_groups)) return SGLC_ERR_ARGUMENT;
-  if (score_fn != 0 && score_fn != 1) return SGLC_ERR_ARGUMENT;
-  return sglc_launch(router_kernel, dim3((T + 63) / 64), dim3(64), 0, stream, 1, true, z, z_stride, correction, dense,
-                     dense_stride, ids, wts, T, E, top, n_groups, keep, renorm, weight_scale, score_fn, renorm_eps);
+  return sglc_router_pass(z, z_stride, correction, dense, dense_stride, ids, wts, T, E, top, n_groups, keep, renorm,
+                          weight_scale, score_fn, renorm_eps, 0, 0, nullptr, stream);
 }
 
 SGLC_API int sglc_router(const float* z, long long z_stride, const float* correction, float* dense,

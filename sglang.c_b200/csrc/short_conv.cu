@@ -171,3 +171,16 @@ SGLC_API int sglc_short_conv(const float* x, long long x_stride, const float* ta
   if (rc != SGLC_OK || K == 1 || p.own_tail) return rc;
   return sglc_launch(short_conv_tail_kernel, dim3(R, (C + 127) / 128), dim3(128), 0, stream, 1, true, p);
 }
+
+// The tails alone: tail[slot] <- the last K-1 inputs of every request after this step's portion, for
+// a convolution that another kernel of the step made (and whose launch ends before this one begins).
+SGLC_API int sglc_short_conv_tail(const float* x, long long x_stride, float* tail, const int* q_start,
+                                  const int* state_slots, int R, int C, int K, int n_slots, int* err,
+                                  cudaStream_t stream) {
+  if (R <= 0 || K <= 1) return SGLC_OK;
+  if (C <= 0 || !tail) return SGLC_ERR_ARGUMENT;
+  ConvArgs p = {};
+  p.x = x; p.x_stride = x_stride; p.tail = tail; p.q_start = q_start; p.state_slots = state_slots;
+  p.R = R; p.C = C; p.K = K; p.n_slots = n_slots; p.err = err;
+  return sglc_launch(short_conv_tail_kernel, dim3(R, (C + 127) / 128), dim3(128), 0, stream, 1, true, p);
+}

@@ -7,18 +7,58 @@ from ..parts.registry import get_part
 from ..weights.loader import DeviceStore, load_checked
 
 
+def _as_tuple(need):
+    return () if need is None else tuple(need) if isinstance(need, (tuple, list)) else (need,)
+
+
 class Layer:
     """A built layer: `block` and the built sub-parts as attributes named by their roles."""
 
     def __init__(self, name, block, parts, mixer_role):
         self.name, self.block, self.parts = name, block, parts
         self.mixer_role = mixer_role
+        self._spans = None
         for role, part in parts.items():
             setattr(self, role, part)
 
     @property
     def the_mixer(self):
         return self.parts[self.mixer_role] if self.mixer_role is not None else None
+
+    def cache_need(self):
+        """What a call of this layer keeps: the mixer's need as it is, or, where other sub-parts keep
+        something too, one tuple of the mixer's needs followed by theirs in the order of the roles."""
+        need = self.the_mixer.cache_need() if self.the_mixer is not None else None
+        others = [p.cache_need() for role, p in self.parts.items() if role != self.mixer_role]
+        others = [n for n in others if n is not None]
+        if not others:
+            return need
+        return _as_tuple(need) + tuple(n for o in others for n in _as_tuple(o))
+
+    def bindings(self, cache):
+        """role -> its binding(s), of what cache_need() asked for (a block with a sub-part beside the
+        mixer that keeps something takes its layer's cache apart with this)."""
+        if self._spans is None:
+            self._spans = self._make_spans()
+        if self._spans == self.mixer_role:
+            return {self.mixer_role: cache}
+        return {role: cache[at] for role, at in self._spans}
+
+    def _make_spans(self):
+        """[(role, its place in the layer's tuple: an index, or a slice)]; the mixer's role alone where
+        only the mixer keeps something."""
+        roles = ([self.mixer_role] if self.mixer_role is not None else []) + \
+            [r for r in self.parts if r != self.mixer_role]
+        asked = [(r, self.parts[r].cache_need()) for r in roles]
+        asked = [(r, n) for r, n in asked if n is not None]
+        if len(asked) == 1 and asked[0][0] == self.mixer_role:
+            return self.mixer_role
+        spans, k = [], 0
+        for role, need in asked:
+            n = len(_as_tuple(need))
+            spans.append((role, slice(k, k + n) if isinstance(need, (tuple, list)) else k))
+            k += n
+        return spans
 
 
 class Model:
@@ -69,8 +109,7 @@ class Model:
 
     def cache_needs(self):
         """(need per call of the running order, cache_of per call)."""
-        mixers = [self.layers[c.layer].the_mixer for c in self.plan.order]
-        needs = [m.cache_need() if m is not None else None for m in mixers]
+        needs = [self.layers[c.layer].cache_need() for c in self.plan.order]
         return needs, [c.cache_of for c in self.plan.order]
 
     def workspace_per_token(self):

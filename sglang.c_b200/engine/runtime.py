@@ -102,29 +102,38 @@ class Runtime:
         ops.attention_simt(q, cache, grp.block_table, ctx.token_req, ctx.positions, out, n_heads,
                            scale, window, ctx.max_keys, max_q_len=ctx.max_q_len)
 
-    def attend_shared(self, ctx, q, binding, grp, out, n_heads, head_dim, scale, window):
+    def attend_shared(self, ctx, q, binding, grp, out, n_heads, head_dim, scale, window, sinks=None, gate=None):
         """Causal attention of the step's queries over a cache whose rows are keys and values at
         once (one shared head: a latent).  The rows of the step's own tokens are in the cache
         already (whoever owns it wrote them).  The same choice of kernel as attend(): single
         tokens to the split-key kernel, prompt portions to the tensor cores where the head size
-        allows, everything else (and the 32-bit path) to the general kernel."""
+        allows, everything else (and the 32-bit path) to the general kernel.  sinks: a score per head that
+        joins the softmax's denominator; gate: pre-activations (one a head, or one an entry) whose sigmoid
+        multiplies the heads' results."""
         cache = binding.tensor
+        plain = sinks is None and gate is None
         bf16_ok = self.dtype == "bfloat16" and head_dim % 8 == 0 and head_dim <= 256 and q.stride(0) % 8 == 0 \
             and q.data_ptr() % 16 == 0
         # single tokens: all heads of a token in one block when the sizes allow (a row is read once,
         # not once per head), else a block per (token, head)
         one_block = bf16_ok and ops.attention_latent_decode_supported(q, cache, n_heads)
         single = ops.attention_latent_decode if one_block else ops.attention_decode_shared
-        if bf16_ok and ctx.max_q_len == 1:
-            return single(q, cache, grp.block_table, None, ctx.positions, out, n_heads, scale, window, ctx.max_keys)
-        if bf16_ok and ops.attention_prefill_tc_supported(q, cache, scale) \
+        more = {} if plain else {"sinks": sinks, "gate": gate}
+        if bf16_ok and ctx.max_q_len == 1 and (plain or one_block):
+            return single(q, cache, grp.block_table, None, ctx.positions, out, n_heads, scale, window, ctx.max_keys, **more)
+        if bf16_ok and ctx.max_q_len > 1 and (plain or one_block) and ops.attention_prefill_tc_supported(q, cache, scale) \
                 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0:
             split = ctx.n_decode > 0
             ops.attention_prefill_tc(q, cache, grp.block_table, ctx.q_start, ctx.kv_len, out, n_heads, scale, window,
-                                     ctx.R, ctx.max_q_len, skip_single=split, kv_shared=True)
+                                     ctx.R, ctx.max_q_len, skip_single=split, kv_shared=True, **more)
             if split:
                 single(q, cache, grp.block_table, ctx.token_req, ctx.positions, out, n_heads, scale, window,
-                       ctx.max_keys, token_list=ctx.decode_tokens, n_tokens=ctx.n_decode)
+                       ctx.max_keys, token_list=ctx.decode_tokens, n_tokens=ctx.n_decode, **more)
+            return
+        if not plain:
+            ops.attention_ext(q, cache, grp.block_table, ctx.token_req, ctx.positions, out, n_heads, 1, head_dim,
+                              head_dim, grp.page_size, scale, window, None, sinks, ctx.max_keys,
+                              max_q_len=ctx.max_q_len, splits=None, kv_shared=True, gate=gate)
             return
         ops.attention_simt(q, cache, grp.block_table, ctx.token_req, ctx.positions, out, n_heads,
                            scale, window, ctx.max_keys, max_q_len=ctx.max_q_len, kv_shared=True)

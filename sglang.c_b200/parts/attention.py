@@ -106,9 +106,13 @@ class LatentAttention(Part):
     [c | k_turned], the absorbed query [Wuk_i^T q_i | q_i_turned]; a head's weighted sum of rows
     carries rot_dim entries that the folded output matrix meets with zero columns.
     `out_mult`: a multiplier of the mixer's result, folded into the output matrix.
+    `sink`: a learned score per head that joins the softmax's denominator once (no row, no value, not
+    scaled).  `gate` "head": head i's result is multiplied by sigmoid(h·Wgᵀ)_i; the gate's rows lie in
+    the product that makes the latents (32-bit), and whoever ends the attention applies it to the
+    weighted sum of rows (the values' and output projections are linear in it).
     params: size, n_heads, qk_dim, v_dim, kv_rank, q_rank (None or a size), scale,
     eps (of the latents' norms), own_latent, window, rot_dim (default 0), rotary (dims, base,
-    pairing, scaling), out_mult (default 1)."""
+    pairing, scaling), out_mult (default 1), sink (default false), gate (None or "head")."""
 
     @classmethod
     def declare_weights(cls, params):
@@ -124,6 +128,12 @@ class LatentAttention(Part):
             d["q_weight"] = WeightDecl((H * (D + Rd), E), "matrix")
         if params.get("own_latent", True):
             d.update({"kv_down": WeightDecl((R + Rd, E), "matrix"), "kv_norm": WeightDecl((R,), "norm_gain")})
+        if params.get("sink"):
+            d["sink"] = WeightDecl((H,), "bias")
+        if params.get("gate"):
+            if params["gate"] != "head":
+                raise ValueError(f"latent attention: gate {params['gate']!r}; known: head")
+            d["gate_weight"] = WeightDecl((H, E), "matrix")
         return d
 
     def load(self, tensors, store):
@@ -147,14 +157,20 @@ class LatentAttention(Part):
             return torch.cat([folded, folded.new_zeros(folded.shape[0], H, Rd)], 2).reshape(-1, H * (R + Rd))
 
         tag = (f",{Rd}" if Rd else "") + (f",*{m!r}" if m != 1.0 else "")
+        self.sink = store.vector(tensors["sink"]) if p.get("sink") else None
+        g = tensors["gate_weight"] if p.get("gate") else None
+        self.gate = None                   # (a product of its own only where no 32-bit product reads h)
         # with a turned part the queries leave their product in 32-bit as well (the turn is 32-bit):
         # direct queries and the latent's projection, which read the same rows, are then one product
         self.q_abs = self.q_and_down = None
         if Rd and not Q and p.get("own_latent", True):
             kv = tensors["kv_down"]
+            extra = [] if g is None else [g]
+            pad = (-(H * (R + Rd) + R + Rd + H)) % 8 if extra else 0
             self.q_and_down = Linear(store.computed(
-                f"fold({k_up.name},{q_src.name}{tag})+{kv.name}",
-                lambda: torch.cat([fold_queries(), kv.tensor.double()], 0)), None)
+                f"fold({k_up.name},{q_src.name}{tag})+" + "+".join(r.name for r in [kv] + extra) + (f"+{pad}" if pad else ""),
+                lambda: torch.cat([fold_queries()] + [r.tensor.double() for r in [kv] + extra] +
+                                  [torch.zeros(pad, kv.tensor.shape[1], dtype=torch.float64)], 0)), None)
         else:
             self.q_abs = Linear(store.computed(f"fold({k_up.name},{q_src.name}{tag})", fold_queries), None)
         self.out = Linear(store.computed(f"fold({w_o.name},{v_up.name}{tag})", fold_output), None)
@@ -177,8 +193,15 @@ class LatentAttention(Part):
         # the projections whose results go through a norm are one product with a 32-bit result
         self.down = None
         if downs and self.q_and_down is None:
-            self.down = Linear(store.computed("+".join(r.name for r in downs),
-                                              lambda: torch.cat([r.tensor.float() for r in downs], 0)), None)
+            pad = 0
+            if g is not None:
+                downs.append(g)
+                pad = (-sum(r.tensor.shape[0] for r in downs)) % 8
+            self.down = Linear(store.computed("+".join(r.name for r in downs) + (f"+{pad}" if pad else ""),
+                                              lambda: torch.cat([r.tensor.float() for r in downs] +
+                                                                [torch.zeros(pad, downs[0].tensor.shape[1])], 0)), None)
+        elif g is not None and self.q_and_down is None:
+            self.gate = Linear(store.matrix(g), None)
 
     def cache_need(self):
         p = self.params
@@ -189,6 +212,8 @@ class LatentAttention(Part):
         act = 4 if self.rt.dtype == "float32" else 2
         W, Q = p["kv_rank"] + int(p.get("rot_dim") or 0), p.get("q_rank") or 0
         turned = 4 * (p["n_heads"] + 1) * W + 1024 if p.get("rot_dim") else 0
+        if p.get("gate"):
+            turned += 4 * p["n_heads"] + 64
         return act * (2 * p["n_heads"] * W + Q) + 4 * (Q + W) + turned
 
     def forward(self, ctx, h, residual, cache, position=None, out=None):
@@ -204,9 +229,13 @@ class LatentAttention(Part):
         if self.rot_dim:
             return self._forward_turned(ctx, h, residual, cache, grp, out)
         q_in = h
+        gate = self._own_gate(ctx, h)
         if self.down is not None:
             low = ctx.alloc((T, self.down.out_size), torch.float32)
             self.down.forward(ctx, h, out=low)
+            if p.get("gate"):
+                n = Q + (R if own else 0)
+                gate = ctx.columns(low, n, n + H)
             if Q:
                 q_in = ctx.alloc((T, Q), self.rt.act_dtype)
                 ops.norm_rows(ctx.columns(low, 0, Q), self.q_norm, None, eps, q_in, form="rms")
@@ -217,8 +246,16 @@ class LatentAttention(Part):
         q = ctx.alloc((T, H * R), self.rt.act_dtype)
         self.q_abs.forward(ctx, q_in, out=q)
         o = ctx.alloc((T, H * R), self.rt.act_dtype)
-        ctx.rt.attend_shared(ctx, q, cache, grp, o, H, R, float(p["scale"]), p.get("window"))
+        ctx.rt.attend_shared(ctx, q, cache, grp, o, H, R, float(p["scale"]), p.get("window"), sinks=self.sink, gate=gate)
         return self.out.forward(ctx, o, out=out, residual=residual)
+
+    def _own_gate(self, ctx, h):
+        """The gate's pre-activations where they come out of a product of their own (else None)."""
+        if self.gate is None:
+            return None
+        z = ctx.alloc((h.shape[0], self.params["n_heads"]), torch.float32)
+        self.gate.forward(ctx, h, out=z)
+        return z
 
     def _forward_turned(self, ctx, h, residual, cache, grp, out):
         """The form with a turned part: queries and the latent's row leave their products in 32-bit;
@@ -231,15 +268,21 @@ class LatentAttention(Part):
         T, W = h.shape[0], R + Rd
         eps = float(p["eps"])
         low = None
+        gate = self._own_gate(ctx, h)
         if self.q_and_down is not None:
-            pre = ctx.alloc((T, H * W + W), torch.float32)
+            pre = ctx.alloc((T, self.q_and_down.out_size), torch.float32)
             self.q_and_down.forward(ctx, h, out=pre)
+            if p.get("gate"):
+                gate = ctx.columns(pre, H * W + W, H * W + W + H)
             qx, low = ctx.columns(pre, 0, H * W), ctx.columns(pre, H * W, H * W + W)
         else:
             q_in = h
             if self.down is not None:
                 lows = ctx.alloc((T, self.down.out_size), torch.float32)
                 self.down.forward(ctx, h, out=lows)
+                if p.get("gate"):
+                    n = Q + (W if own else 0)
+                    gate = ctx.columns(lows, n, n + H)
                 if Q:
                     q_in = ctx.alloc((T, Q), self.rt.act_dtype)
                     ops.norm_rows(ctx.columns(lows, 0, Q), self.q_norm, None, eps, q_in, form="rms")
@@ -252,7 +295,7 @@ class LatentAttention(Part):
         ops.latent_rope(qx, low, self.kv_norm, eps, ctx.positions, rot.frequencies, rot.multiplier, rot.dims,
                         rot.pairing, q, cache.tensor.view(-1, W) if own else None, grp.slots, H, R, Rd)
         o = ctx.alloc((T, H * W), self.rt.act_dtype)
-        ctx.rt.attend_shared(ctx, q, cache, grp, o, H, W, float(p["scale"]), p.get("window"))
+        ctx.rt.attend_shared(ctx, q, cache, grp, o, H, W, float(p["scale"]), p.get("window"), sinks=self.sink, gate=gate)
         return self.out.forward(ctx, o, out=out, residual=residual)
 
 
@@ -348,9 +391,19 @@ class RotaryAttention(Part):
     projections have biases.  `own_kv` false: the layer has no key and value projections (nor
     `k_norm`) and reads what another call cached (the plan's `cache_of`).  `out_mult`: a multiplier
     of the mixer's result (the values are cached times it: the attention is linear in them).
+    `sink` "one": a constant 1 in the softmax's denominator (a sink whose score is 0) instead of a
+    learned score.  `gate` "entry": the heads' results, side by side, are multiplied entry by entry by
+    sigmoid(h·Wgᵀ) ahead of the output projection; whoever ends the attention does it, in 32-bit.
+    `temp`: a learned factor per head of its scores (not of the sink); with "row_gain" it is part of
+    the queries' gain.  `conv`: the projected channels of q, k and v pass a causal convolution of so
+    many taps over time (no activation, no bias) ahead of norm and turn, in the input stage's launch;
+    the last conv - 1 projected values are kept per request, 32-bit, also by a layer that reads
+    another's keys (for its queries).  `cache_chunk`: the chunk by which the cache may give pages back,
+    where a call with another chunk reads them too (default: `chunk`).
     params: size, n_heads, n_kv_heads, head_dim, v_dim, scale, rotary (dims, base, scaling, pairing) or
-    None, qk_norm, eps, chunk, window, sink, bias (default false), own_kv (default true), out_mult
-    (default 1)."""
+    None, qk_norm, eps, chunk, window, sink (false, true or "one"), bias (default false), own_kv (default
+    true), out_mult (default 1), gate (None or "entry"), temp (default false), conv (default None),
+    cache_chunk."""
 
     @classmethod
     def declare_weights(cls, params):
@@ -367,8 +420,21 @@ class RotaryAttention(Part):
             d["q_norm"] = WeightDecl((D if norm == "head_gain" else H * D,), "norm_gain")
             if own:
                 d["k_norm"] = WeightDecl((D if norm == "head_gain" else G * D,), "norm_gain")
-        if params.get("sink"):
+        if params.get("sink") and params["sink"] != "one":
             d["sink"] = WeightDecl((H,), "bias")
+        if params.get("gate"):
+            if params["gate"] != "entry":
+                raise ValueError(f"rotary_attention: gate {params['gate']!r}; known: entry")
+            d["gate_weight"] = WeightDecl((H * V, E), "matrix")
+        if params.get("temp"):
+            if norm != "row_gain":
+                raise ValueError("rotary_attention: a factor per head goes with qk_norm \"row_gain\"")
+            d["temp"] = WeightDecl((H,), "norm_gain")
+        if params.get("conv"):
+            d["q_conv"] = WeightDecl((H * D, params["conv"]), "conv_taps")
+            if own:
+                d["k_conv"] = WeightDecl((G * D, params["conv"]), "conv_taps")
+                d["v_conv"] = WeightDecl((G * V, params["conv"]), "conv_taps")
         return d
 
     def load(self, tensors, store):
@@ -378,13 +444,17 @@ class RotaryAttention(Part):
         self.mult = float(p.get("out_mult", 1.0))
         roles = ("q", "k", "v") if self.own else ("q",)
         refs = [tensors[k + "_weight"] for k in roles]
+        self.channels = sum(r.tensor.shape[0] for r in refs)
+        if p.get("gate"):
+            refs.append(tensors["gate_weight"])
         n = sum(r.tensor.shape[0] for r in refs)
         pad = (-n) % 8
         bias = None
         if p.get("bias", False):
             brefs = [tensors[k + "_bias"] for k in roles]
-            bias = store.computed("+".join(r.name for r in brefs) + f"+{pad}", kind="vector", make=lambda: torch.cat(
-                [r.tensor.float() for r in brefs] + [torch.zeros(pad)]))
+            zeros = n + pad - self.channels                # (a gate has no bias)
+            bias = store.computed("+".join(r.name for r in brefs) + f"+{zeros}", kind="vector", make=lambda: torch.cat(
+                [r.tensor.float() for r in brefs] + [torch.zeros(zeros)]))
         self.qkv = Linear(store.computed("+".join(r.name for r in refs) + f"+{pad}", lambda: torch.cat(
             [r.tensor.float() for r in refs] + [torch.zeros(pad, refs[0].tensor.shape[1])], 0)), bias)
         out_bias = None
@@ -393,20 +463,38 @@ class RotaryAttention(Part):
             out_bias = store.vector(ob) if m == 1.0 else store.computed(
                 f"{ob.name}*{m!r}", kind="vector", make=lambda: (ob.tensor.double() * m).float())
         self.out = Linear(store.matrix(tensors["out_weight"]), out_bias)
-        self.sink = store.vector(tensors["sink"]) if p.get("sink") else None
+        self.sink = None
+        if p.get("sink") == "one":
+            self.sink = store.computed(f"zeros:{p['n_heads']}", kind="vector", make=lambda: torch.zeros(p["n_heads"]))
+        elif p.get("sink"):
+            self.sink = store.vector(tensors["sink"])
+        self.taps = None
+        if p.get("conv"):                  # [taps, channels]: a tap's channels lie side by side
+            crefs = [tensors[k + "_conv"] for k in roles]
+            self.taps = store.computed("+".join(r.name for r in crefs) + ".T", kind="vector", make=lambda: torch.cat(
+                [r.tensor.float() for r in crefs], 0).t())
         rot = p.get("rotary") or {"dims": 0, "base": 10000.0, "scaling": None}
         self.rotary = get_part("position", "rotary")(rot, self.rt)
         self.rotary.load({}, store)
         self.norm = p.get("qk_norm")
         self.q_gain = store.vector(tensors["q_norm"]) if "q_norm" in tensors else None
         self.k_gain = store.vector(tensors["k_norm"]) if "k_norm" in tensors else None
+        if p.get("temp"):
+            g, tp = tensors["q_norm"], tensors["temp"]
+            self.q_gain = store.computed(f"{g.name}*{tp.name}", kind="vector", make=lambda: (
+                g.tensor.double().view(p["n_heads"], -1) * tp.tensor.double()[:, None]).reshape(-1))
         # the first kernel of this mixer serves its first form: unit-RMS heads behind a turn of halves
         self.general = self.norm in ("head_gain", "row_gain") or self.rotary.pairing != "halves" or not self.own \
-            or self.mult != 1.0
+            or self.mult != 1.0 or self.taps is not None
 
     def cache_need(self):
         p = self.params
-        return CacheNeed.paged_kv(p["n_kv_heads"], p["head_dim"], p.get("window"), v_dim=p["v_dim"], chunk=p.get("chunk"))
+        H, G, D, V = p["n_heads"], p["n_kv_heads"], p["head_dim"], p["v_dim"]
+        kv = CacheNeed.paged_kv(G, D, p.get("window"), v_dim=V, chunk=p.get("cache_chunk", p.get("chunk")))
+        if not p.get("conv"):
+            return kv
+        channels = H * D + (G * (D + V) if p.get("own_kv", True) else 0)
+        return kv, CacheNeed.state((p["conv"] - 1, channels), "float32", private=True)
 
     def workspace_per_token(self):
         p = self.params
@@ -414,13 +502,17 @@ class RotaryAttention(Part):
         act = 4 if self.rt.dtype == "float32" else 2
         from ..csrc import ops
         # (a step of single tokens deals a token's keys to several blocks: their shares)
-        return 4 * ((H + G) * D + G * V + 8) + act * H * (D + V) + 1024 + 4 * H * ops.EXT_MAX_SPLITS * (V + 2)
+        gate = H * V if p.get("gate") else 0
+        return 4 * ((H + G) * D + G * V + gate + 8) + act * H * (D + V) + 1024 + 4 * H * ops.EXT_MAX_SPLITS * (V + 2)
 
     def forward(self, ctx, h, residual, cache, position=None, out=None):
         from ..csrc import ops
         p = self.params
         H, G, D, V = p["n_heads"], p["n_kv_heads"], p["head_dim"], p["v_dim"]
         T = h.shape[0]
+        tail = None
+        if self.taps is not None:
+            cache, tail = cache
         grp = ctx.group(cache.group)
         if self.own != cache.write:
             raise ValueError("rotary_attention: a layer with key and value projections owns its cache, one "
@@ -433,12 +525,15 @@ class RotaryAttention(Part):
             ops.qk_prep(ctx.columns(pre, 0, H * D + Gown * (D + V)), ctx.positions, self.rotary.frequencies,
                         self.rotary.multiplier, self.rotary.dims, self.rotary.pairing, self.norm, float(p["eps"]),
                         self.q_gain, self.k_gain, q, cache.tensor if self.own else None,
-                        grp.slots if self.own else None, H, Gown, D, V, grp.page_size, v_mult=self.mult)
+                        grp.slots if self.own else None, H, Gown, D, V, grp.page_size, v_mult=self.mult,
+                        conv=None if tail is None else (self.taps, tail.tensor, ctx.token_req, ctx.q_start,
+                                                        ctx.state_slots, ctx.R))
         else:
             ops.rotary_kv(ctx.columns(pre, 0, (H + G) * D + G * V), ctx.positions, self.rotary.frequencies,
                           self.rotary.multiplier, self.rotary.dims, float(p["eps"]) if p.get("qk_norm") else None, q,
                           cache.tensor, grp.slots, H, G, D, V, grp.page_size)
         o = ctx.alloc((T, H * V), self.rt.act_dtype)
+        gate = ctx.columns(pre, self.channels, self.channels + H * V) if p.get("gate") else None
         # a step of prompt portions only, keys and values of one size the tensor-core kernel takes (a
         # page is then its [2][G][page_size][D]): 128-query tiles on the tensor cores; every other
         # step (single tokens among them, other sizes, 32-bit) goes to the general kernel
@@ -446,7 +541,7 @@ class RotaryAttention(Part):
             pages = cache.tensor.view(cache.tensor.shape[0], 2, G, grp.page_size, D)
             if ops.attention_prefill_tc_supported(q, pages, float(p["scale"])) and o.stride(0) % 8 == 0:
                 ops.attention_prefill_tc(q, pages, grp.block_table, ctx.q_start, ctx.kv_len, o, H, float(p["scale"]),
-                                         p.get("window"), ctx.R, ctx.max_q_len, chunk=p.get("chunk"), sinks=self.sink)
+                                         p.get("window"), ctx.R, ctx.max_q_len, chunk=p.get("chunk"), sinks=self.sink, gate=gate)
                 return self.out.forward(ctx, o, out=out, residual=residual)
         # every other step goes to the general kernel; where every request brings one token, a
         # token's keys are dealt to several blocks and a second launch merges their shares
@@ -454,7 +549,7 @@ class RotaryAttention(Part):
         ws = ctx.alloc((T * H * splits * (V + 2),), torch.float32) if splits > 1 else None
         ops.attention_ext(q, cache.tensor, grp.block_table, ctx.token_req, ctx.positions, o, H, G, D, V, grp.page_size,
                           float(p["scale"]), p.get("window"), p.get("chunk"), self.sink, ctx.max_keys,
-                          max_q_len=ctx.max_q_len, splits=splits, workspace=ws)
+                          max_q_len=ctx.max_q_len, splits=splits, workspace=ws, gate=gate)
         return self.out.forward(ctx, o, out=out, residual=residual)
 
 

@@ -22,6 +22,9 @@ Interfaces by category (ctx is an `engine.step.StepContext`):
                                                  residual += ff(h), or out = ff(h)
   stream_mix    begin(ctx, x) / finish(ctx, x)   around a layer: x becomes a mix of this and
                                                  earlier layers' results (kept in ctx.shared)
+  token_mix     forward(ctx, x, norm1, h1, norm2, h2, cache)
+                                                 h1 = norm1(x) mixed with earlier tokens' (kept in
+                                                 `cache`), h2 = norm2(x) (or norm2, h2 None)
   block         forward(ctx, x, layer, cache, position)
                                                  runs norm1/mixer/norm2/ffn of `layer` on x
   head          forward(ctx, h, out)             out[W,V] float32 logits of h[W,E]
@@ -55,6 +58,7 @@ class Part:
         parts name."""
 
     def cache_need(self):
+        """What the part keeps per request (mixers, and parts of category token_mix)."""
         return None
 
     def workspace_per_token(self, *args):

@@ -113,6 +113,48 @@ class ParallelSublayersBlock(Part):
         return x
 
 
+@register_part("block", "parallel_two_norms")
+class ParallelTwoNormsBlock(Part):
+    """A norm for each of two parallel sublayers: x += mixer(norm1(x)) + ffn(norm2(x)), both of the
+    same x; the feed-forward is there only if the layer has an `ffn`.  With a `shift` sub-part (category
+    token_mix) what the mixer reads is first mixed with the tokens before.  Both norms (RMS, one eps,
+    no biases) and the shift are one launch, so the sublayers' last products may add into the 32-bit
+    stream from their epilogues as each ends."""
+
+    def workspace_per_token(self, layer):
+        act = 4 if self.rt.dtype == "float32" else 2
+        inner = layer.mixer.workspace_per_token()
+        if "ffn" in layer.parts:
+            inner = max(inner, layer.ffn.workspace_per_token())
+        return 2 * act * layer.norm1.params["size"] + 512 + inner
+
+    def forward(self, ctx, x, layer, cache, position=None):
+        from ..csrc import ops
+        T, E = x.shape
+        mark = ctx.mark()
+        has_ffn = "ffn" in layer.parts
+        norms = [layer.norm1] + ([layer.norm2] if has_ffn else [])
+        for n in norms:
+            if n.form != "rms" or n.bias is not None or n.groups != 1 or n.params["eps"] != layer.norm1.params["eps"]:
+                raise ValueError("parallel_two_norms: two plain RMS norms with one eps")
+        h1 = ctx.alloc((T, E), self.rt.act_dtype)
+        h2 = ctx.alloc((T, E), self.rt.act_dtype) if has_ffn else None
+        norm2 = layer.norm2 if has_ffn else None
+        kept = layer.bindings(cache)
+        if "shift" in layer.parts:
+            layer.shift.forward(ctx, x, layer.norm1, h1, norm2, h2, kept["shift"])
+        else:
+            ops.norm_pair_shift(x, layer.norm1.weight, norm2.weight if has_ffn else None,
+                                float(layer.norm1.params["eps"]), h1, h2)
+        inner = ctx.mark()
+        layer.mixer.forward(ctx, h1, residual=x, cache=kept.get("mixer"), position=position)
+        ctx.release(inner)
+        if has_ffn:
+            layer.ffn.forward(ctx, h2, residual=x)
+        ctx.release(mark)
+        return x
+
+
 @register_part("block", "post_norm")
 class PostNormBlock(Part):
     """A norm on each sublayer's result only; the sublayers read the stream itself:

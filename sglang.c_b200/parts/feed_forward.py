@@ -137,16 +137,21 @@ class RoutedExperts(Part):
     sigmoid), `renorm` (the chosen scores divided by their sum + 1e-20), `weight_scale` (a factor
     of every weight), `correction` false (no such tensor).  `shared_inner_size`: one more expert of
     that inner width (`shared_gate`, `shared_up`, `shared_down`) that every token uses with weight
-    1; its matrices lie behind the routed experts' in the same two products.
+    1; its matrices lie behind the routed experts' in the same two products.  `n_identity`: the router
+    chooses among so many more experts, behind the n_experts (scores, correction and groups count them
+    too), that have no tensors and hand h on as it is; their share w h is formed by the gating's launch.
+    `group_score` "max": a group scores its largest choice score.
     params: size, inner_size (an expert's), n_experts, top, n_groups, keep, score, renorm,
-    weight_scale, correction, shared_inner_size."""
+    weight_scale, correction, shared_inner_size, n_identity, group_score ("top2_sum", the default, or
+    "max")."""
 
     @classmethod
     def declare_weights(cls, params):
         E, F, X = params["size"], params["inner_size"], params["n_experts"]
-        d = {"router": WeightDecl((X, E), "matrix")}
+        Xr = X + int(params.get("n_identity") or 0)          # the router's outputs
+        d = {"router": WeightDecl((Xr, E), "matrix")}
         if params.get("correction", True):
-            d["correction"] = WeightDecl((X,), "bias")
+            d["correction"] = WeightDecl((Xr,), "bias")
         for e in range(X):
             d.update({f"gate_{e}": WeightDecl((F, E), "matrix"), f"up_{e}": WeightDecl((F, E), "matrix"),
                       f"down_{e}": WeightDecl((E, F), "residual_matrix")})
@@ -166,7 +171,7 @@ class RoutedExperts(Part):
         self.down = Linear(store.computed("|".join(r.name for r in downs),
                                           lambda: torch.cat([r.tensor.float() for r in downs], 1)), None)
         rw = tensors["router"]
-        pad = (-X) % 8
+        pad = (-(X + int(self.params.get("n_identity") or 0))) % 8
         self.router = Linear(store.computed(rw.name + f"+{pad}", lambda: torch.cat(
             [rw.tensor.float(), torch.zeros(pad, rw.tensor.shape[1])], 0)), None)
         self.correction = store.vector(tensors["correction"]) if "correction" in tensors else None
@@ -175,7 +180,8 @@ class RoutedExperts(Part):
         p = self.params
         act = 4 if self.rt.dtype == "float32" else 2
         X = p["n_experts"]
-        return act * 3 * (X * p["inner_size"] + int(p.get("shared_inner_size") or 0)) + 4 * (2 * X + 8) + 8 * p["top"] + 1024
+        Xr = X + int(p.get("n_identity") or 0)
+        return act * 3 * (X * p["inner_size"] + int(p.get("shared_inner_size") or 0)) + 4 * (2 * Xr + 9) + 8 * p["top"] + 1024
 
     def forward(self, ctx, h, residual, out=None):
         from ..csrc import ops
@@ -183,16 +189,26 @@ class RoutedExperts(Part):
         T, F, X, top = h.shape[0], p["inner_size"], p["n_experts"], p["top"]
         z = ctx.alloc((T, self.router.out_size), torch.float32)
         self.router.forward(ctx, h, out=z)
-        dense = ctx.alloc((T, X), torch.float32)
+        n_id = int(p.get("n_identity") or 0)
+        dense = ctx.alloc((T, X + n_id), torch.float32)
+        passed = ctx.alloc((T,), torch.float32) if n_id else None
         ids = ctx.alloc((T, top), torch.int32)
         wts = ctx.alloc((T, top), torch.float32)
         renorm = bool(p.get("renorm", False))
-        ops.router(ctx.columns(z, 0, X), self.correction, dense, ids, wts, top, p.get("n_groups", 1), p.get("keep", 1),
+        ops.router(ctx.columns(z, 0, X + n_id), self.correction, dense, ids, wts, top, p.get("n_groups", 1), p.get("keep", 1),
                    renorm=renorm, weight_scale=float(p.get("weight_scale", 1.0)), score=p.get("score", "sigmoid"),
-                   renorm_eps=1e-20 if renorm else 0.0)
+                   renorm_eps=1e-20 if renorm else 0.0, group_score=p.get("group_score", "top2_sum"), n_pass=n_id,
+                   handed_on=passed)
         Fall = X * F + int(p.get("shared_inner_size") or 0)      # the shared expert's columns take weight 1
         gu = ctx.alloc((T, 2 * Fall), self.rt.act_dtype)
         self.gate_up.forward(ctx, h, out=gu)
         a = ctx.alloc((T, Fall), self.rt.act_dtype)
-        ops.gated_act(gu, a, weights=dense, per=F, n_weighted=X * F)
-        return self.down.forward(ctx, a, out=out, residual=residual)
+        if not n_id:
+            ops.gated_act(gu, a, weights=dense, per=F, n_weighted=X * F)
+            return self.down.forward(ctx, a, out=out, residual=residual)
+        # the identity experts' share goes into the stream (or begins the result), the products add to it
+        add = residual is not None
+        dst = residual if add else out
+        ops.gated_act(gu, a, weights=ctx.columns(dense, 0, X), per=F, n_weighted=X * F,
+                      handed_on=(h, passed, dst[:T], add))
+        return self.down.forward(ctx, a, residual=dst)

@@ -43,8 +43,8 @@ class LayerPlan:
     the block's business: the pre-norm block asks for norm1, mixer, norm2, ffn; another block may
     ask for one norm beside a mixer and a feed-forward, or for a pair of norms behind them.
     `parts` maps role -> (category, PartSpec); the four usual roles can also be given (and later
-    replaced) as attributes.  A layer has at most one sub-part of category "mixer": its cache
-    need is the layer's."""
+    replaced) as attributes.  A layer has at most one sub-part of category "mixer": what
+    it keeps per request is the layer's (other sub-parts may keep something beside it)."""
 
     def __init__(self, name, block, norm1=None, mixer=None, norm2=None, ffn=None, parts=None):
         object.__setattr__(self, "name", name)

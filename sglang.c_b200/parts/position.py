@@ -67,10 +67,13 @@ class RotaryPositions(PositionEncoding):
     which `original` positions make t turns, lo = max(floor(pair(fast)), 0), hi = min(ceil(pair(slow)),
     dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency is
     f_i / factor * ramp_i + f_i (1 - ramp_i), and cos and sin are both multiplied by
-    0.1 ln(factor) + 1.  The table is made once, in 64-bit; the mixer's kernel forms the angles.
+    0.1 ln(factor) + 1.  With `scaling` = {factor, original, low, high} (the rule of Llama 3.1) a pair
+    keeps f_i if more than `high` of its wavelengths 2 pi / f_i fit into `original` positions, takes
+    f_i / factor if fewer than `low` do, and between the two, with t of them fitting and s = (t - low)
+    / (high - low), takes (1 - s) f_i / factor + s f_i; no multiplier.  The table is made once, in 64-bit; the mixer's kernel forms the angles.
     A mixer builds this part from its own params (a model may turn each layer differently).
     `pairing` "neighbours" pairs entry 2i with 2i+1 instead (for the kernels that take the choice).
-    params: dims, base, scaling (None or the four numbers), pairing ("halves", the default, or
+    params: dims, base, scaling (None or the four numbers of either rule), pairing ("halves", the default, or
     "neighbours")."""
 
     def load(self, tensors, store):
@@ -81,7 +84,12 @@ class RotaryPositions(PositionEncoding):
         i = torch.arange(dims // 2, dtype=torch.float64)
         f = base ** (-2.0 * i / dims) if dims else i
         self.multiplier = 1.0
-        if sc and dims:
+        if sc and dims and "high" in sc:
+            factor, low, high = float(sc["factor"]), float(sc["low"]), float(sc["high"])
+            turns = float(sc["original"]) * f / (2.0 * math.pi)
+            s = ((turns - low) / (high - low)) if high != low else torch.zeros_like(f)
+            f = torch.where(turns > high, f, torch.where(turns < low, f / factor, (1.0 - s) * f / factor + s * f))
+        elif sc and dims:
             factor, orig = float(sc["factor"]), float(sc["original"])
             pair = lambda turns: dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
             lo = max(math.floor(pair(float(sc["fast"]))), 0)
