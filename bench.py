@@ -18,7 +18,7 @@ requests) over its time, against the measured copy bandwidth; `points` has decod
 at batch 1 and 64, the true 32-bit path and the prefill through the C interface;
 `kernels` says where a decode and a
 prefill step's time goes, kernel by kernel.  `--full` adds medium and XL layer
-sizes and the mixed workload to `points`.  `--compare tukavik` (or `zuretar`, or `buborax`, each of which adds its design as one more column; `lubavik`: that design beside Zuretar, the closest one) measures,
+sizes and the mixed workload to `points`.  `--compare tukavik` (or `zuretar`, or `buborax`, each of which adds its design as one more column; `lubavik`: that design beside Zuretar, the closest one; `fupapel`: that design beside Lubavik, the closest, and Tukavik for its latents) measures,
 instead of all this, a Tukavik model beside the GPT-2 model of the same layer sizes.
 """
 import argparse
@@ -904,6 +904,68 @@ def lubavik_step_bytes(cfg, batch, context, prompt_tokens):
     return out
 
 
+def fupapel_config(base, n_layer):
+    """A Fupapel model with the layer sizes of a GPT-2 model: the same width, depth, head size (64) and
+    vocabulary.  Layers in fours: chunked attention behind convolutions of four taps (the model's heads
+    over a quarter as many key/value heads, chunks of 320, scaled rotation); latent attention (the model's
+    heads of 64 plus 32 turned entries over a latent of 96, so a cached row of 128; queries through a
+    latent of half the width); chunked attention with gated results (the same heads and chunks); and the
+    first kind again with the first layer's keys and values.  Every layer has a mixture of 8 experts of a
+    sixth of GPT-2's inner width and 2 identity experts, 2 chosen out of one of two groups."""
+    E, H, I = base["n_embd"], base["n_head"], base["n_inner"]
+    moe = {"kind": "moe", "expert": {"ff": max(64, (I // 6) // 64 * 64)},
+           "router": {"experts": 8, "top": 2, "identity": 2, "groups": {"count": 2, "keep": 1}}}
+    chunked = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": 320}}
+    conv = dict(chunked, conv=4, rot={"base": 10000.0, "dims": 64,
+                                      "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 256}})
+    latent = {"heads": H, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 96, "q_rank": E // 2, "scale": 96 ** -0.5,
+              "rot": {"base": 10000.0, "dims": 32}}
+    layers = []
+    for i in range(n_layer):
+        kind, m = [("attention_2", conv), ("latent_attention", latent),
+                   ("attention", dict(chunked, rot={"base": 10000.0, "dims": 32})),
+                   ("attention_2", dict(conv, kv_from=i - 3))][i % 4]
+        layers.append({"type": kind, "mixer": m, "mlp": moe})
+    return {"architecture": "Fupapel", "vocab": base["vocab_size"], "width": E, "norm": {"eps": 1e-6},
+            "residual_mult": 0.4, "layers": layers, "max_positions": base["n_positions"]}
+
+
+def fupapel_step_bytes(cfg, batch, context, prompt_tokens):
+    """What the kernels that this design adds or extends must move in a step (32-bit projections and
+    states; bfloat16 activations and cache): {decode | prefill: {kernel label: bytes}}."""
+    E = cfg["width"]
+    out = {}
+    for name, T, R in (("decode", batch, batch), ("prefill", prompt_tokens, 2)):
+        prep = rope = attn = latent = gact = route = pair = tails = 0
+        for layer in cfg["layers"]:
+            m = layer["mixer"]
+            pair += T * E * (4 + 2 + 2) + R * E * 8            # the stream, both norms' rows, the rows kept
+            if layer["type"] == "latent_attention":
+                W = m["kv_rank"] + m["rot_dim"]
+                rope += T * (m["heads"] + 1) * W * (4 + 2)
+                if name == "decode":
+                    latent += T * context * W * 2 + T * m["heads"] * W * 4
+            else:
+                H, D, V = m["heads"], m["dim"], m["vdim"]
+                G = 0 if "kv_from" in m else m["kv_heads"]
+                C = H * D + G * (D + V)
+                prep += T * C * (4 + 2)
+                if "conv" in m:
+                    state = R * (m["conv"] - 1) * C * 8
+                    prep += state if name == "decode" else 0
+                    tails += state
+                if name == "decode":
+                    seen = context % m["mask"]["size"]
+                    attn += T * seen * m["kv_heads"] * (D + V) * 2 + T * H * (D + V) * 2
+            r = layer["mlp"]["router"]
+            F = layer["mlp"]["expert"]["ff"] * r["experts"]
+            gact += T * F * 6 + T * E * (8 + 2) * 2 // 10       # (a fifth of the tokens' choices are identities)
+            route += T * (r["experts"] + r["identity"]) * 8 + T * r["top"] * 8
+        out[name] = {"norm_pair_shift": pair, "qk_prep": prep, "short_conv_tail": tails, "latent_rope": rope,
+                     "attention_ext": attn, "attention_latent_decode": latent, "gated_act": gact, "router": route}
+    return out
+
+
 DESIGNS = {"tukavik": (tukavik_config, tukavik_step_bytes,
                        {"mingru_scan": "mingru_scan", "norm_rows": "norm_rows", "depth_mix": "depth_mix",
                         "attention_decode_shared": "attention_shared"}),
@@ -914,7 +976,10 @@ DESIGNS = {"tukavik": (tukavik_config, tukavik_step_bytes,
                                        "gated_act", "norm_rows", "cast_rows")}),
            "lubavik": (lubavik_config, lubavik_step_bytes,
                        {k: k for k in ("qk_prep", "matrix_state", "stabilized_gates", "gated_norm", "attention_ext",
-                                       "gated_act", "norm_add_tail", "gated_gather", "router")})}
+                                       "gated_act", "norm_add_tail", "gated_gather", "router")}),
+           "fupapel": (fupapel_config, fupapel_step_bytes,
+                       {k: k for k in ("norm_pair_shift", "qk_prep", "short_conv_tail", "latent_rope", "attention_ext",
+                                       "attention_latent_decode", "gated_act", "router")})}
 
 
 def compare_designs(designs, sizes, steps, warmup, pk):
@@ -1043,7 +1108,7 @@ def main():
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "fp32"],
                     help="a handful of steps of one kind and nothing else (what a profiler is pointed at): "
                          "decode steps at batch 8, prefill steps of 2 x 1,024 tokens, or both on the 32-bit path")
-    ap.add_argument("--compare", default=None, choices=["tukavik", "zuretar", "buborax", "lubavik"],
+    ap.add_argument("--compare", default=None, choices=["tukavik", "zuretar", "buborax", "lubavik", "fupapel"],
                     help="nothing of the above: decode and prefill of a model of this design beside the GPT-2 model "
                          "of equal layer sizes (--model, or small and medium with --full), with both kernel tables")
     args = ap.parse_args()
@@ -1064,7 +1129,8 @@ def main():
         clocks = ClockSampler()
         clocks.start()
         designs = {"tukavik": ["tukavik"], "zuretar": ["tukavik", "zuretar"],
-                   "buborax": ["tukavik", "zuretar", "buborax"], "lubavik": ["zuretar", "lubavik"]}[args.compare]
+                   "buborax": ["tukavik", "zuretar", "buborax"], "lubavik": ["zuretar", "lubavik"],
+                   "fupapel": ["tukavik", "lubavik", "fupapel"]}[args.compare]
         res = compare_designs(designs, ["small", "medium"] if args.full else [args.model], steps, warmup, pk)
         print(json.dumps({"metric": f"decode and prefill tok/s, {' and '.join(d.capitalize() for d in designs)} beside "
                                     "GPT-2 at equal layer sizes (Python engine)",

@@ -221,6 +221,8 @@ latent_merge_kernel(LatentArgs a) {
   const float* w = a.ws + ((size_t)slot_t * a.n_splits * H + h) * (D + 2);
   const size_t step = (size_t)H * (D + 2);
   float m[MAX_SPLITS], l[MAX_SPLITS], v[MAX_SPLITS];
+  const float z = a.gate ? a.gate[(size_t)t * a.gate_stride + (a.gate_per_head ? h : i)] : 0.0f;
+  const float sk = a.sinks ? a.sinks[h] : -INFINITY;
 #pragma unroll
   for (int sp = 0; sp < MAX_SPLITS; sp++) {
     const bool on = sp < a.n_splits;
@@ -228,10 +230,10 @@ latent_merge_kernel(LatentArgs a) {
     l[sp] = on ? w[sp * step + D + 1] : 0.0f;
     v[sp] = on ? w[sp * step + d] : 0.0f;
   }
-  float M = a.sinks ? a.sinks[h] : -INFINITY;
+  float M = sk;
 #pragma unroll
   for (int sp = 0; sp < MAX_SPLITS; sp++) M = fmaxf(M, m[sp]);
-  float L = a.sinks ? expf(a.sinks[h] - M) : 0.0f, o = 0.0f;
+  float L = a.sinks ? expf(sk - M) : 0.0f, o = 0.0f;
 #pragma unroll
   for (int sp = 0; sp < MAX_SPLITS; sp++) {
     const float f = l[sp] > 0.0f ? expf(m[sp] - M) : 0.0f;      // (a range past the token's keys is empty)
@@ -239,7 +241,7 @@ latent_merge_kernel(LatentArgs a) {
     o = fmaf(v[sp], f, o);
   }
   o /= L;
-  if (a.gate) o *= gate_of(a, t, h, d);
+  if (a.gate) o *= 1.0f / (1.0f + expf(-z));
   a.out[(size_t)t * a.o_stride + i] = __float2bfloat16_rn(o);
 }
 }  // namespace
@@ -252,10 +254,10 @@ SGLC_API int sglc_attention_latent_decode_supports(int H, int D) {
   return smem <= 200 * 1024;
 }
 
-// Key ranges for T tokens with up to max_keys keys: enough blocks to fill the SMs, a range no
-// shorter than one tile.
+// Key ranges for T tokens with up to max_keys keys: enough blocks to fill the SMs several times over
+// (three of them share an SM), a range no shorter than one tile.
 SGLC_API int sglc_attention_latent_decode_splits(int T, int max_keys) {
-  int want = (148 + T - 1) / T;
+  int want = (512 + T - 1) / T;
   const int most = (max_keys + KT - 1) / KT;
   if (want > most) want = most;
   if (want > MAX_SPLITS) want = MAX_SPLITS;

@@ -273,7 +273,7 @@ static int attention_simt_run(const void* q, int q_stride, const void* cache,
   const int W = single ? 1 : 8;
   const size_t smem = ((size_t)32 * (D % 4 == 0 ? D + 4 : D + 1) + (size_t)32 * DV + (size_t)W * D + (size_t)W * 32) * sizeof(float);
   if (smem > 224 * 1024) return SGLC_ERR_UNSUPPORTED;
-  if (part_ws && (!ext || !single || n_splits < 1 || n_splits > 65535)) return SGLC_ERR_ARGUMENT;
+  if (part_ws && (!ext || !single || n_splits < 1 || n_splits > 32)) return SGLC_ERR_ARGUMENT;
   dim3 grid((T + W - 1) / W, H, part_ws ? n_splits : 1);
   // single tokens whose shares are merged afterwards: where 2 to 8 query heads share a key/value
   // head, a block takes them all (the eight-warp form, its warps being heads of one token)
@@ -393,23 +393,27 @@ attention_merge_kernel(const float* __restrict__ part_ws, int n_splits, const fl
   if (item >= (long long)T * H) return;
   const int t = (int)(item / H), h = (int)(item % H);
   const float* rec = part_ws + (size_t)item * n_splits * (DV + 2);
-  float M = sinks ? sinks[h] : -INFINITY;
-  for (int s = 0; s < n_splits; s++)
-    if (rec[(size_t)s * (DV + 2) + 1] > 0.0f) M = fmaxf(M, rec[(size_t)s * (DV + 2)]);
-  float L = sinks ? expf(sinks[h] - M) : 0.0f;
-  for (int s = 0; s < n_splits; s++) {
-    const float ls = rec[(size_t)s * (DV + 2) + 1];
-    if (ls > 0.0f) L += ls * expf(rec[(size_t)s * (DV + 2)] - M);
-  }
-  const float inv = 1.0f / L;
+  // lane s holds share s's maximum and sum (an empty share: -inf and 0, its results zero)
+  const float ms = lane < n_splits ? rec[(size_t)lane * (DV + 2)] : -INFINITY;
+  const float ls = lane < n_splits ? rec[(size_t)lane * (DV + 2) + 1] : 0.0f;
+  const float sk = sinks ? sinks[h] : -INFINITY;
+  const float z_head = gate.z && gate.per_head ? gate.z[t * gate.stride + h] : 0.0f;
+  const float M = fmaxf(warp_max(ls > 0.0f ? ms : -INFINITY), sk);
+  const float f = ls > 0.0f ? expf(ms - M) : 0.0f;
+  const float L = warp_sum(ls * f) + (sinks ? expf(sk - M) : 0.0f);
+  float inv = 1.0f / L;
+  if (gate.z && gate.per_head) inv *= 1.0f / (1.0f + expf(-z_head));
+  const bool by_entry = gate.z && !gate.per_head;
   TO* op = out + (size_t)t * o_stride + (size_t)h * DV;
-  for (int d = lane; d < DV; d += 32) {
+  for (int d0 = 0; d0 < DV; d0 += 32) {
+    const int d = d0 + lane;
+    const float z = by_entry && d < DV ? gate.z[t * gate.stride + (long long)h * DV + d] : 0.0f;
     float o = 0.0f;
     for (int s = 0; s < n_splits; s++)
-      if (rec[(size_t)s * (DV + 2) + 1] > 0.0f) o += rec[(size_t)s * (DV + 2) + 2 + d] * expf(rec[(size_t)s * (DV + 2)] - M);
+      o = fmaf(d < DV ? rec[(size_t)s * (DV + 2) + 2 + d] : 0.0f, __shfl_sync(0xffffffffu, f, s), o);
     o *= inv;
-    if (gate.z) o *= out_gate(gate, t, h, DV, d);
-    op[d] = from_f32<TO>(o);
+    if (by_entry) o *= 1.0f / (1.0f + expf(-z));
+    if (d < DV) op[d] = from_f32<TO>(o);
   }
 }
 

@@ -111,14 +111,39 @@ struct PassRows {
   const float* w;                         // [rows]
   float* x; long long x_stride;
   int E, add;
+  int first_block;                        // the launch's blocks from here on do this and nothing else
+  int by4;                                // four columns a thread (E, the strides and the addresses allow it)
 };
+__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
 template <typename TI>
 __device__ __forceinline__ void pass_rows(const PassRows& p, int rows) {
-  if (!p.h) return;
   const TI* h = static_cast<const TI*>(p.h);
-  const long long total = (long long)rows * p.E;
-  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
-       i += (long long)gridDim.x * blockDim.x) {
+  const long long first = (long long)(blockIdx.x - p.first_block) * blockDim.x + threadIdx.x;
+  const long long step = (long long)(gridDim.x - p.first_block) * blockDim.x;
+  if (p.by4) {
+    const int E4 = p.E / 4;
+    for (long long i = first; i < (long long)rows * E4; i += step) {
+      const long long r = i / E4;
+      const int c = (int)(i % E4) * 4;
+      const float w = p.w[r];
+      const float4 v = four(h + r * p.h_stride + c);
+      float4* xp = reinterpret_cast<float4*>(p.x + r * p.x_stride + c);
+      if (!p.add) {
+        *xp = make_float4(w * v.x, w * v.y, w * v.z, w * v.w);
+      } else if (w != 0.0f) {
+        const float4 o = *xp;
+        *xp = make_float4(fmaf(w, v.x, o.x), fmaf(w, v.y, o.y), fmaf(w, v.z, o.z), fmaf(w, v.w, o.w));
+      }
+    }
+    return;
+  }
+  for (long long i = first; i < (long long)rows * p.E; i += step) {
     const long long r = i / p.E;
     const int c = (int)(i % p.E);
     const float w = p.w[r];
@@ -134,10 +159,10 @@ __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_strid
                                  const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
-  pass_rows<TO>(pass, rows);
+  if ((int)blockIdx.x >= pass.first_block) return pass_rows<TO>(pass, rows);
   const long long total = (long long)rows * F;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
-       i += (long long)gridDim.x * blockDim.x) {
+       i += (long long)pass.first_block * blockDim.x) {
     const long long r = i / F;
     const int c = (int)(i % F);
     const float wt = (w && c < n_weighted) ? w[r * w_stride + c / per] : 1.0f;
@@ -158,11 +183,11 @@ __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, lon
                                       int n_weighted, const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
-  pass_rows<__nv_bfloat16>(pass, rows);
+  if ((int)blockIdx.x >= pass.first_block) return pass_rows<__nv_bfloat16>(pass, rows);
   const int F8 = F / 8;
   const long long total = (long long)rows * F8;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
-       i += (long long)gridDim.x * blockDim.x) {
+       i += (long long)pass.first_block * blockDim.x) {
     const long long r = i / F8;
     const int c = (int)(i % F8) * 8;
     const float wt = ((w && c < n_weighted) ? w[r * w_stride + c / per] : 1.0f) * mult;
@@ -189,23 +214,33 @@ __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, lon
 // n_weighted: the first so many columns (a multiple of `per`) take weights, the rest take 1
 static int gated_act_run(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
                          int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
-                         int act, float mult, int n_weighted, const PassRows& pass, cudaStream_t stream) {
+                         int act, float mult, int n_weighted, PassRows pass, cudaStream_t stream) {
   if (rows <= 0 || F <= 0) return SGLC_OK;
   if (act != GA_SILU && act != GA_GELU_TANH) return SGLC_ERR_ARGUMENT;
   if (w && (per <= 0 || n_weighted < 0 || n_weighted > F || n_weighted % per != 0)) return SGLC_ERR_ARGUMENT;
   const long long total = (long long)rows * F;
   int blocks = (int)((total + 255) / 256);
   if (blocks > 148 * 16) blocks = 148 * 16;
+  int more = 0;                                // blocks for the rows handed on
+  if (pass.h) {
+    const int bytes = dst_dtype == SGLC_F32 ? 16 : 8;
+    pass.by4 = pass.E % 4 == 0 && pass.h_stride % 4 == 0 && pass.x_stride % 4 == 0 && ((uintptr_t)pass.x & 15) == 0 &&
+               ((uintptr_t)pass.h & (bytes - 1)) == 0;
+    const long long n = (long long)rows * pass.E / (pass.by4 ? 4 : 1);
+    more = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+  }
+  pass.first_block = blocks;
   if (src_dtype == SGLC_BF16 && dst_dtype == SGLC_BF16 && F % 8 == 0 && src_stride % 8 == 0 && dst_stride % 8 == 0 &&
       (!w || (per % 8 == 0 && n_weighted % 8 == 0)) && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0) {
     int b8 = (int)((total / 8 + 255) / 256);
     if (b8 > 148 * 16) b8 = 148 * 16;
-    return sglc_launch(gated_act_vec8_kernel, dim3(b8), dim3(256), 0, stream, 1, true, (const __nv_bfloat16*)src,
+    pass.first_block = b8;
+    return sglc_launch(gated_act_vec8_kernel, dim3(b8 + more), dim3(256), 0, stream, 1, true, (const __nv_bfloat16*)src,
                        src_stride, (__nv_bfloat16*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult,
                        n_weighted, pass);
   }
 #define LAUNCH(TI, TO)                                                                                  \
-  return sglc_launch(gated_act_kernel<TI, TO>, dim3(blocks), dim3(256), 0, stream, 1, true, (const TI*)src, \
+  return sglc_launch(gated_act_kernel<TI, TO>, dim3(blocks + more), dim3(256), 0, stream, 1, true, (const TI*)src, \
                      src_stride, (TO*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult, n_weighted, pass)
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_F32) LAUNCH(float, float);
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_BF16) LAUNCH(float, __nv_bfloat16);
@@ -229,7 +264,7 @@ SGLC_API int sglc_gated_act_pass(const void* src, long long src_stride, int src_
                                  const float* w_pass, float* x, long long x_stride, int E, int add,
                                  cudaStream_t stream) {
   if (!h || !w_pass || !x || E <= 0) return SGLC_ERR_ARGUMENT;
-  PassRows pass = {h, h_stride, w_pass, x, x_stride, E, add};
+  PassRows pass = {h, h_stride, w_pass, x, x_stride, E, add, 0, 0};
   return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per, act, mult,
                        n_weighted, pass, stream);
 }

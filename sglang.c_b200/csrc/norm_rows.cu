@@ -449,6 +449,80 @@ __global__ void norm_pair_shift_kernel(const float* __restrict__ x, const float*
   }
 }
 
+// The same for steps of many tokens (four floats at a time): a block takes PAIR_TOKENS consecutive
+// tokens, a warp each, and one warp more for the token ahead of them, so a row is read once by a block
+// that needs it twice.  A portion's first token finds its slot and its portion's last row by itself.
+constexpr int PAIR_TOKENS = 8;
+
+template <typename TO>
+__global__ void __launch_bounds__((PAIR_TOKENS + 1) * 32)
+norm_pair_shift_rows_kernel(const float* __restrict__ x, const float* __restrict__ g1, const float* __restrict__ g2,
+                            const float* __restrict__ mu, float eps, float* __restrict__ prev,
+                            const int* __restrict__ token_req, const int* __restrict__ q_start,
+                            const int* __restrict__ state_slots, TO* __restrict__ y1, long long y1_stride,
+                            TO* __restrict__ y2, long long y2_stride, int T, int E, int n_slots, int* __restrict__ err) {
+  extern __shared__ __align__(16) float rows[];   // [PAIR_TOKENS + 1][E]
+  __shared__ float inv_s[PAIR_TOKENS + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * PAIR_TOKENS + warp - 1;      // (warp 0: the token ahead of the block's)
+  pdl_launch_dependents();
+  bool head = false;
+  int last = t, slot = -1;
+  if (mu && warp > 0 && t < T) {
+    const int r = token_req[t];
+    head = t == q_start[r];
+    last = q_start[r + 1] - 1;
+    slot = state_slots[r];
+  }
+  pdl_wait();
+  const int n_it = E / 4;
+  float4* mine = reinterpret_cast<float4*>(rows + (size_t)warp * E);
+  if (t >= 0 && t < T && (warp > 0 || mu)) {
+    float q = 0.0f;
+    for (int i = lane; i < n_it; i += 32) {
+      const float4 v = reinterpret_cast<const float4*>(x + (size_t)t * E)[i];
+      mine[i] = v;
+      q = sq4(v, 0.0f, q);
+    }
+    q = warp_sum(q);
+    if (lane == 0) inv_s[warp] = 1.0f / sqrtf(q / (float)E + eps);
+  }
+  __syncthreads();
+  if (warp == 0 || t >= T) return;
+  const float ia = inv_s[warp];
+  float ib = warp > 0 ? inv_s[warp - 1] : 0.0f;
+  const float4* before = reinterpret_cast<const float4*>(rows + (size_t)(warp - 1) * E);
+  float4* ps = nullptr;
+  if (head) {
+    if (!sglc_index_ok(slot, n_slots, err)) return;
+    ps = reinterpret_cast<float4*>(prev + (size_t)slot * E);
+    before = reinterpret_cast<const float4*>(x + (size_t)last * E);      // what the slot takes
+    float q = 0.0f;
+    for (int i = lane; i < n_it; i += 32) q = sq4(before[i], 0.0f, q);
+    ib = 1.0f / sqrtf(warp_sum(q) / (float)E + eps);
+  }
+  TO* o1 = y1 + (size_t)t * y1_stride;
+  TO* o2 = y2 ? y2 + (size_t)t * y2_stride : nullptr;
+  for (int i = lane; i < n_it; i += 32) {
+    const float4 v = mine[i];
+    float4 h = norm4(v, 0.0f, ia, g1, nullptr, i);
+    if (mu) {
+      const float4 hb = norm4(before[i], 0.0f, ib, g1, nullptr, i);
+      float4 p = hb;
+      if (head) {
+        p = ps[i];
+        ps[i] = hb;
+      }
+      const float4 m = reinterpret_cast<const float4*>(mu)[i];
+      h = make_float4(fmaf(p.x - h.x, m.x, h.x), fmaf(p.y - h.y, m.y, h.y), fmaf(p.z - h.z, m.z, h.z),
+                      fmaf(p.w - h.w, m.w, h.w));
+    }
+    store4<TO>(o1 + 4 * i, h);
+    if (o2) store4<TO>(o2 + 4 * i, norm4(v, 0.0f, ia, g2, nullptr, i));
+  }
+}
+constexpr int PAIR_ROWS_MIN = 296;      // tokens from which the form above is used: two blocks' worth of rows an SM
+
 // x: float [T][E] contiguous; g1, g2, mu: float [E] (g2 with y2 only; mu may be null); prev: float
 // [n_slots][E] (with mu); y1, y2 (y2 may be null): [T][stride] of out_dtype.
 SGLC_API int sglc_norm_pair_shift(const float* x, const float* g1, const float* g2, const float* mu, float eps,
@@ -465,6 +539,20 @@ SGLC_API int sglc_norm_pair_shift(const float* x, const float* g1, const float* 
   const bool vec = E % 4 == 0 && al16(x) && al16(g1) && al16(g2) && al16(mu) && al16(prev) && y1_stride % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(y1) & oa) == 0 &&
                    (!y2 || (y2_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(y2) & oa) == 0));
+  const size_t smem_rows = (size_t)(PAIR_TOKENS + 1) * E * sizeof(float);
+  if (vec && T >= PAIR_ROWS_MIN && smem_rows <= 100 * 1024) {
+    const dim3 grid((T + PAIR_TOKENS - 1) / PAIR_TOKENS), block((PAIR_TOKENS + 1) * 32);
+#define ROWS(TO)                                                                                                  \
+  do {                                                                                                            \
+    if (smem_rows > 48 * 1024)                                                                                    \
+      cudaFuncSetAttribute(norm_pair_shift_rows_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_rows); \
+    return sglc_launch(norm_pair_shift_rows_kernel<TO>, grid, block, smem_rows, stream, 1, true, x, g1, g2, mu, eps, prev, \
+                       token_req, q_start, state_slots, (TO*)y1, y1_stride, (TO*)y2, y2_stride, T, E, n_slots, err); \
+  } while (0)
+    if (out_dtype == SGLC_BF16) ROWS(__nv_bfloat16);
+    ROWS(float);
+#undef ROWS
+  }
 #define PAIR(TO, VEC)                                                                                            \
   do {                                                                                                           \
     if (smem > 48 * 1024)                                                                                        \

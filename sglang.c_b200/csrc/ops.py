@@ -1167,12 +1167,17 @@ def gated_gather(z, tokens, table, first, dst, err_flag=None):
 EXT_MAX_SPLITS = 16         # blocks a token's keys are dealt to at most (attention_ext in a step of single tokens)
 
 
-def attention_ext_splits(max_keys, window=None, chunk=None):
+def attention_ext_splits(max_keys, window=None, chunk=None, n_blocks=None):
     """How many blocks share a token's keys in a step of single tokens: two tiles of 32 keys a block,
-    up to EXT_MAX_SPLITS (1: the plain launch)."""
+    up to EXT_MAX_SPLITS (1: the plain launch).  n_blocks: the launch's blocks without the split (tokens times
+    key/value heads): no more shares than keep all blocks resident at once."""
     seen = min(int(max_keys), int(window or max_keys), int(chunk or max_keys))
     tiles = (seen + 31) // 32 + 1
-    return max(1, min(EXT_MAX_SPLITS, tiles // 2))
+    most = EXT_MAX_SPLITS if n_blocks is None else max(1, EXT_RESIDENT_BLOCKS // int(n_blocks))
+    return max(1, min(EXT_MAX_SPLITS, tiles // 2, most))
+
+
+EXT_RESIDENT_BLOCKS = 3 * 148
 
 
 def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_kv_heads, dim, v_dim, page_size,
@@ -1182,8 +1187,8 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
     [n_pages, G*page_size*(dim+v_dim)]: a page's keys, then its values), an optional chunk mask
     (a query sees the keys of its own chunk of `chunk` positions) and an optional sink per head
     (float32 [H]) in the softmax's denominator.  q [T, H*dim]; out [T, H*v_dim].
-    splits > 1 (a step of single tokens only): every token's keys are dealt to so many blocks, whose
-    shares a second launch merges; workspace: float32, T * H * splits * (v_dim + 2) entries.
+    splits > 1, or a workspace (a step of single tokens only): every token's keys are dealt to so many blocks
+    (one: all query heads of a key/value head together), whose shares a second launch merges; workspace: float32, T * H * splits * (v_dim + 2) entries.
     kv_shared: the cache keeps one row of `dim` entries per position and head, a key whose first v_dim
     entries are its value.  splits None: chosen here, with the library's own scratch.  gate: float32 pre-activations [T, H] or [T, H*v_dim] whose sigmoid
     multiplies the heads' results."""
@@ -1205,9 +1210,11 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
         splits = 1
         if max_q_len == 1:
             workspace = _tc_buffers(q.device)[0]
-            splits = min(attention_ext_splits(max_keys, window, chunk), workspace.numel() // (T * n_heads * (v_dim + 2)))
-            splits = max(splits, 1)
-    if splits > 1:
+            splits = min(attention_ext_splits(max_keys, window, chunk, T * n_kv_heads),
+                         workspace.numel() // (T * n_heads * (v_dim + 2)))
+            if splits < 1:
+                splits, workspace = 1, None
+    if splits > 1 or workspace is not None:
         if (max_q_len or 2) > 1 or workspace is None or workspace.dtype != torch.float32 \
                 or workspace.numel() < T * n_heads * splits * (v_dim + 2) or not workspace.is_contiguous():
             raise KernelError("attention_ext: keys are split over blocks in a step of single tokens only, with a "
@@ -1278,33 +1285,49 @@ ROUTER_MAX_EXPERTS = 256
 
 
 def router(logits, correction, dense, ids, weights, top, n_groups=1, keep=1, renorm=False, weight_scale=1.0,
-           score="sigmoid", renorm_eps=0.0, group_score="top2_sum", n_pass=0, handed_on=None):
+           score="sigmoid", renorm_eps=0.0, group_score="top2_sum", n_pass=0, handed_on=None, rows=None, matrix=None):
     """Routing by sigmoid scores (or, score "softmax", a softmax over all experts) with a choice
     correction and group limits; renorm: the chosen scores divided by their sum + renorm_eps; then
     times weight_scale (see router.cu).  logits: float32
     [T, E]; correction: float32 [E] or None; dense: float32 [T, E] (weights, zero where not
     chosen); ids int32 [T, top]; weights float32 [T, top].  group_score: "top2_sum", or "max" (a group
     counts as its best expert).  handed_on (float32 [T]): takes the sum of a token's weights for the
-    last n_pass experts."""
-    _need_cuda(logits, correction, dense, ids, weights, handed_on)
+    last n_pass experts.  logits None: they are made in the same launch, rows [T, K] times matrix
+    [>= E, K] (its first E rows), both of one dtype, summed in 32-bit."""
+    _need_cuda(logits, correction, dense, ids, weights, handed_on, rows, matrix)
     T, E = dense.shape
-    _f32_rows(logits, "router: logits", E)
     _f32_rows(dense, "router: dense", E)
     if ids.dtype != torch.int32 or not ids.is_contiguous() or tuple(ids.shape) != (T, top) \
             or weights.dtype != torch.float32 or not weights.is_contiguous() or tuple(weights.shape) != (T, top):
         raise KernelError("router: ids int32 [T, top], weights float32 [T, top]")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
         raise KernelError("router: one float32 correction per expert")
-    lib = build.load("router")
     if handed_on is not None and (handed_on.dtype != torch.float32 or handed_on.numel() < T
                                   or not handed_on.is_contiguous()):
         raise KernelError("router: handed_on is float32 [T]")
-    code = lib.sglc_router_pass(_ptr(logits), ctypes.c_longlong(logits.stride(0)), _ptr(correction), _ptr(dense),
-                               ctypes.c_longlong(dense.stride(0)), _ptr(ids), _ptr(weights), T, E, int(top),
-                               int(n_groups), int(keep), 1 if renorm else 0, ctypes.c_float(weight_scale),
-                               {"sigmoid": 0, "softmax": 1}[score], ctypes.c_float(renorm_eps),
-                               {"top2_sum": 0, "max": 1}[group_score], int(n_pass), _ptr(handed_on), _stream())
+    lib = build.load("router")
+    tail = (_ptr(correction), _ptr(dense), ctypes.c_longlong(dense.stride(0)), _ptr(ids), _ptr(weights), T, E, int(top),
+            int(n_groups), int(keep), 1 if renorm else 0, ctypes.c_float(weight_scale), {"sigmoid": 0, "softmax": 1}[score],
+            ctypes.c_float(renorm_eps), {"top2_sum": 0, "max": 1}[group_score], int(n_pass), _ptr(handed_on), _stream())
+    if logits is None:
+        if rows.dtype != matrix.dtype or rows.shape[0] < T or rows.stride(1) != 1 or not matrix.is_contiguous() \
+                or matrix.shape[0] < E or matrix.shape[1] != rows.shape[1]:
+            raise KernelError("router: rows [T, K] and matrix [>= E, K] of one dtype")
+        code = lib.sglc_router_product(_ptr(rows), ctypes.c_longlong(rows.stride(0)), _ptr(matrix), rows.shape[1],
+                                       _dt(rows, "router rows"), *tail)
+    else:
+        _f32_rows(logits, "router: logits", E)
+        code = lib.sglc_router_pass(_ptr(logits), ctypes.c_longlong(logits.stride(0)), *tail)
     _check(lib, code, f"router ({E} experts, {top} chosen)")
+
+
+# a router's matrix is re-read by every token of the fused form: what a step may re-read (from L2) before a
+# product of its own is the cheaper way
+ROUTER_PRODUCT_BYTES = 8 << 20
+
+
+def router_product_pays(n_tokens, matrix):
+    return n_tokens * matrix.numel() * matrix.element_size() <= ROUTER_PRODUCT_BYTES
 
 
 def cast_rows(src, dst):

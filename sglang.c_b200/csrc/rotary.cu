@@ -19,6 +19,11 @@ SGLC_DEFINE_ERROR_STRING()
 constexpr int ROT_WARPS = 4;
 constexpr int ROT_MAX_DIM = 512;
 
+// (u, v) -> (u cos a - v sin a, v cos a + u sin a), with the roundings written out: which of the two
+// products is the fused one is then the same in every kernel
+__device__ __forceinline__ float turn_u(float u, float v, float cs, float sn) { return fmaf(u, cs, -__fmul_rn(v, sn)); }
+__device__ __forceinline__ float turn_v(float u, float v, float cs, float sn) { return fmaf(v, cs, __fmul_rn(u, sn)); }
+
 template <typename TA>
 __global__ void __launch_bounds__(ROT_WARPS * 32)
 rotary_kv_kernel(const float* __restrict__ x, long long x_stride, const int* __restrict__ positions,
@@ -114,9 +119,18 @@ latent_rope_kernel(const float* __restrict__ qx, long long qx_stride, const floa
                    int H, int R, int Rd, int* err) {
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  pdl_wait();
-  const int pos = positions[t];
+  const int pos = positions[t];                // (the step's own array: no kernel of the step writes it)
   const int half = dims / 2, W = R + Rd;
+  extern __shared__ float2 turn[];             // (cosine, sine) of the token's pairs, made once for all rows
+  for (int i = threadIdx.x; i < half; i += ROT_WARPS * 32) {
+    double a = (double)pos * freq[i];
+    a -= floor(a * 0.15915494309189535) * 6.283185307179586;
+    float sn, cs;
+    sincosf((float)a, &sn, &cs);
+    turn[i] = make_float2(cs * mult, sn * mult);
+  }
+  pdl_wait();
+  __syncthreads();
   for (int row = warp; row < H + (low ? 1 : 0); row += ROT_WARPS) {
     const float* src;
     TA* dst;
@@ -138,15 +152,11 @@ latent_rope_kernel(const float* __restrict__ qx, long long qx_stride, const floa
     src += R;
     dst += R;
     for (int i = lane; i < half; i += 32) {
-      double a = (double)pos * freq[i];
-      a -= floor(a * 0.15915494309189535) * 6.283185307179586;
-      float sn, cs;
-      sincosf((float)a, &sn, &cs);
-      sn *= mult; cs *= mult;
+      const float cs = turn[i].x, sn = turn[i].y;
       const int iu = pairing ? 2 * i : i, iv = pairing ? 2 * i + 1 : i + half;
       const float u = src[iu], v = src[iv];
-      dst[iu] = from_f32<TA>(u * cs - v * sn);
-      dst[iv] = from_f32<TA>(v * cs + u * sn);
+      dst[iu] = from_f32<TA>(turn_u(u, v, cs, sn));
+      dst[iv] = from_f32<TA>(turn_v(u, v, cs, sn));
     }
     for (int d = 2 * half + lane; d < Rd; d += 32) dst[d] = from_f32<TA>(src[d]);
   }
@@ -163,11 +173,11 @@ SGLC_API int sglc_latent_rope(const float* qx, long long qx_stride, const float*
   if (H <= 0 || R <= 0 || Rd < 0 || dims < 0 || dims > Rd || dims % 2 != 0 || (low && (!gain || !rows || !slots)))
     return SGLC_ERR_ARGUMENT;
   if (dtype == SGLC_F32)
-    return sglc_launch(latent_rope_kernel<float>, dim3(T), dim3(ROT_WARPS * 32), 0, stream, 1, true, qx, qx_stride, low,
+    return sglc_launch(latent_rope_kernel<float>, dim3(T), dim3(ROT_WARPS * 32), (size_t)dims / 2 * sizeof(float2), stream, 1, true, qx, qx_stride, low,
                        low_stride, gain, eps, positions, freq, mult, dims, pairing, (float*)q_out, q_stride, (float*)rows,
                        slots, n_rows, T, H, R, Rd, err);
   if (dtype == SGLC_BF16)
-    return sglc_launch(latent_rope_kernel<__nv_bfloat16>, dim3(T), dim3(ROT_WARPS * 32), 0, stream, 1, true, qx,
+    return sglc_launch(latent_rope_kernel<__nv_bfloat16>, dim3(T), dim3(ROT_WARPS * 32), (size_t)dims / 2 * sizeof(float2), stream, 1, true, qx,
                        qx_stride, low, low_stride, gain, eps, positions, freq, mult, dims, pairing,
                        (__nv_bfloat16*)q_out, q_stride, (__nv_bfloat16*)rows, slots, n_rows, T, H, R, Rd, err);
   return SGLC_ERR_ARGUMENT;
@@ -196,13 +206,18 @@ SGLC_API int sglc_latent_rope(const float* qx, long long qx_stride, const float*
 // (short_conv.cu: short_conv_tail_kernel), when nobody reads a tail any more.
 constexpr int QK_WARPS = 8;      // (a token's head rows are dealt to the warps: eight keep the rounds few)
 
+__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
 struct QkConv {
   const float* taps;              // [K][C], C = H*D + G*(D+V)
   float* tail;                    // [n_slots][K-1][C]
   const int* token_req;           // [T]
   const int* q_start;             // [R+1]
   const int* state_slots;         // [R]
-  int K, n_slots, own_tail;
+  int K, n_slots, own_tail, by4;  // by4: four channels a thread (C, the stride and the addresses allow it)
 };
 
 template <typename TA, bool CONV>
@@ -211,40 +226,70 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
                const double* __restrict__ freq, float mult, int dims, int pairing, int norm_mode, float eps,
                const float* __restrict__ gain_q, const float* __restrict__ gain_k, float v_mult,
                TA* __restrict__ q_out, long long q_stride, TA* __restrict__ cache, const int* __restrict__ slots,
-               int T, int H, int G, int D, int V, int page_size, int n_pages, int* err, const QkConv cv) {
+               int T, int H, int G, int D, int V, int page_size, int n_pages, int* err, const QkConv cv, int by2) {
   __shared__ float buf[QK_WARPS][ROT_MAX_DIM];
   __shared__ float red[2][QK_WARPS];
+  __shared__ float2 turn[ROT_MAX_DIM / 2];     // (cosine, sine) of the token's pairs, made once for all its heads
   extern __shared__ __align__(16) float conv_row[];      // CONV: the token's convolved channels
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  pdl_wait();
+  // (positions and slots are the step's own arrays: no kernel of the step writes them)
   const int pos = positions[t];
   const int slot = G > 0 ? slots[t] : -1;
   const int page = slot / page_size, off = slot % page_size;
   const bool page_ok = G > 0 && slot >= 0 && sglc_index_ok(page, n_pages, err);
   const size_t page_elems = (size_t)G * page_size * (D + V);
   const float* xr = x + (size_t)t * x_stride;
+  for (int i = threadIdx.x; i < dims / 2; i += QK_WARPS * 32) {
+    double a = (double)pos * freq[i];
+    a -= floor(a * 0.15915494309189535) * 6.283185307179586;
+    float sn, cs;
+    sincosf((float)a, &sn, &cs);
+    turn[i] = make_float2(cs * mult, sn * mult);
+  }
   if constexpr (CONV) {
     const int C = H * D + G * (D + V), K = cv.K;
     const int r = cv.token_req[t], i = t - cv.q_start[r], slot_r = cv.state_slots[r];
     if (!sglc_index_ok(slot_r, cv.n_slots, err)) return;
     float* tail = cv.tail + (size_t)slot_r * (K - 1) * C;
-    for (int ch = threadIdx.x; ch < C; ch += QK_WARPS * 32) {
-      float acc = 0.0f;
-      for (int j = 0; j < K; j++) {
-        const int back = K - 1 - j;            // the input so many tokens ago
-        const float v = back <= i ? xr[ch - (long long)back * x_stride] : tail[(size_t)(K - 1 + i - back) * C + ch];
-        acc = fmaf(cv.taps[(size_t)j * C + ch], v, acc);
+    pdl_wait();
+    if (cv.by4) {
+      for (int ch = threadIdx.x * 4; ch < C; ch += QK_WARPS * 32 * 4) {
+        float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int j = 0; j < K; j++) {
+          const int back = K - 1 - j;          // the input so many tokens ago
+          const float4 v = *reinterpret_cast<const float4*>(
+              back <= i ? xr + ch - (long long)back * x_stride : tail + (size_t)(K - 1 + i - back) * C + ch);
+          const float4 w = *reinterpret_cast<const float4*>(cv.taps + (size_t)j * C + ch);
+          acc = make_float4(fmaf(w.x, v.x, acc.x), fmaf(w.y, v.y, acc.y), fmaf(w.z, v.z, acc.z), fmaf(w.w, v.w, acc.w));
+        }
+        *reinterpret_cast<float4*>(conv_row + ch) = acc;
+        if (cv.own_tail && K > 1) {            // (ascending: an entry is read before its place is written)
+          for (int m = 0; m + 1 < K - 1; m++)
+            *reinterpret_cast<float4*>(tail + (size_t)m * C + ch) = *reinterpret_cast<float4*>(tail + (size_t)(m + 1) * C + ch);
+          *reinterpret_cast<float4*>(tail + (size_t)(K - 2) * C + ch) = *reinterpret_cast<const float4*>(xr + ch);
+        }
       }
-      conv_row[ch] = acc;
-      if (cv.own_tail && K > 1) {              // (ascending: an entry is read before its place is written)
-        for (int m = 0; m + 1 < K - 1; m++) tail[(size_t)m * C + ch] = tail[(size_t)(m + 1) * C + ch];
-        tail[(size_t)(K - 2) * C + ch] = xr[ch];
+    } else {
+      for (int ch = threadIdx.x; ch < C; ch += QK_WARPS * 32) {
+        float acc = 0.0f;
+        for (int j = 0; j < K; j++) {
+          const int back = K - 1 - j;
+          const float v = back <= i ? xr[ch - (long long)back * x_stride] : tail[(size_t)(K - 1 + i - back) * C + ch];
+          acc = fmaf(cv.taps[(size_t)j * C + ch], v, acc);
+        }
+        conv_row[ch] = acc;
+        if (cv.own_tail && K > 1) {
+          for (int m = 0; m + 1 < K - 1; m++) tail[(size_t)m * C + ch] = tail[(size_t)(m + 1) * C + ch];
+          tail[(size_t)(K - 2) * C + ch] = xr[ch];
+        }
       }
     }
-    __syncthreads();
     xr = conv_row;
+  } else {
+    pdl_wait();
   }
+  __syncthreads();
   const int half = dims / 2;
   float inv_all[2] = {1.0f, 1.0f};
   if (norm_mode == 3) {
@@ -261,6 +306,52 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
     for (int w = 0; w < QK_WARPS; w++) { sq += red[0][w]; sk += red[1][w]; }
     inv_all[0] = 1.0f / sqrtf(sq / (float)(H * D) + eps);
     if (G > 0) inv_all[1] = 1.0f / sqrtf(sk / (float)(G * D) + eps);
+  }
+  if ((norm_mode == 0 || norm_mode == 3) && by2) {
+    // no head has statistics of its own: the token's entries lie flat before the block, two a thread and
+    // load (and the two they are paired with).  Units: the turned pairs of the query and key heads, their
+    // passing entries, the values.
+    const int h2 = half / 2, p2 = (D - dims) / 2, n_turn = (H + G) * h2, n_pass = (H + G) * p2;
+    TA* qt = q_out + (size_t)t * q_stride;
+    TA* kt = G > 0 ? cache + (size_t)page * page_elems + (size_t)off * D : nullptr;
+    for (int unit = threadIdx.x; unit < n_turn + n_pass + G * V / 2; unit += QK_WARPS * 32) {
+      if (unit >= n_turn + n_pass) {
+        const int e = (unit - n_turn - n_pass) * 2, g = e / V, d = e % V;
+        if (page_ok) {
+          const float2 v = *reinterpret_cast<const float2*>(xr + (size_t)(H + G) * D + e);
+          store2(cache + (size_t)page * page_elems + (size_t)G * page_size * D + ((size_t)g * page_size + off) * V + d,
+                 v.x * v_mult, v.y * v_mult);
+        }
+        continue;
+      }
+      const bool turned = unit < n_turn;
+      const int row = turned ? unit / h2 : (unit - n_turn) / p2;
+      const int d = turned ? unit % h2 * 2 : dims + (unit - n_turn) % p2 * 2;
+      const bool is_q = row < H;
+      const float* src = xr + (size_t)row * D + d;
+      TA* dst = is_q ? qt + (size_t)row * D + d : page_ok ? kt + (size_t)(row - H) * page_size * D + d : nullptr;
+      const float* gn = norm_mode == 3 ? (is_q ? gain_q + (size_t)row * D : gain_k + (size_t)(row - H) * D) + d : nullptr;
+      const float inv = inv_all[is_q ? 0 : 1];
+      auto take = [&](int at) {
+        float2 v = *reinterpret_cast<const float2*>(src + at);
+        if (gn) {
+          const float2 g = *reinterpret_cast<const float2*>(gn + at);
+          v = make_float2(__fmul_rn(__fmul_rn(v.x, inv), g.x), __fmul_rn(__fmul_rn(v.y, inv), g.y));
+        }
+        return v;
+      };
+      const float2 u = take(0);
+      if (!turned) {
+        if (dst) store2(dst, u.x, u.y);
+        continue;
+      }
+      const float2 v = take(half), c0 = turn[d], c1 = turn[d + 1];
+      if (dst) {
+        store2(dst, turn_u(u.x, v.x, c0.x, c0.y), turn_u(u.y, v.y, c1.x, c1.y));
+        store2(dst + half, turn_v(u.x, v.x, c0.x, c0.y), turn_v(u.y, v.y, c1.x, c1.y));
+      }
+    }
+    return;
   }
   float* b = buf[warp];
   for (int row = warp; row < H + 2 * G; row += QK_WARPS) {
@@ -294,14 +385,10 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
     __syncwarp();
     ss = 0.0f;
     for (int i = lane; i < half; i += 32) {
-      double a = (double)pos * freq[i];
-      a -= floor(a * 0.15915494309189535) * 6.283185307179586;
-      float sn, cs;
-      sincosf((float)a, &sn, &cs);
-      sn *= mult; cs *= mult;
+      const float cs = turn[i].x, sn = turn[i].y;
       const int iu = pairing ? 2 * i : i, iv = pairing ? 2 * i + 1 : i + half;
       const float u = b[iu], v = b[iv];
-      const float ru = u * cs - v * sn, rv = v * cs + u * sn;
+      const float ru = turn_u(u, v, cs, sn), rv = turn_v(u, v, cs, sn);
       b[iu] = ru; b[iv] = rv;
       ss = fmaf(ru, ru, fmaf(rv, rv, ss));
     }
@@ -342,16 +429,21 @@ static int qk_prep_run(const float* x, long long x_stride, const int* positions,
     cv = *conv;
     if (cv.K < 1 || !cv.taps || !cv.token_req || !cv.q_start || !cv.state_slots || (cv.K > 1 && !cv.tail))
       return SGLC_ERR_ARGUMENT;
-    smem = ((size_t)H * D + (size_t)G * (D + V)) * sizeof(float);
+    const long long C = (long long)H * D + (long long)G * (D + V);
+    cv.by4 = C % 4 == 0 && x_stride % 4 == 0 && (((uintptr_t)x | (uintptr_t)cv.taps | (uintptr_t)cv.tail) & 15) == 0;
+    smem = (size_t)C * sizeof(float);
     if (smem > 200 * 1024) return SGLC_ERR_UNSUPPORTED;
   }
+  // pairs of entries side by side: even sizes and halves, addresses that allow two floats a load
+  const int by2 = pairing == 0 && dims % 4 == 0 && D % 2 == 0 && V % 2 == 0 && x_stride % 2 == 0 && q_stride % 2 == 0 &&
+                  (((uintptr_t)x | (uintptr_t)gain_q | (uintptr_t)gain_k | (uintptr_t)q_out | (uintptr_t)cache) & 7) == 0;
 #define PREP(TA, CV)                                                                                               \
   do {                                                                                                             \
     if (smem > 24 * 1024)                                                                                          \
       cudaFuncSetAttribute(qk_prep_kernel<TA, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
     return sglc_launch(qk_prep_kernel<TA, CV>, dim3(T), dim3(QK_WARPS * 32), smem, stream, 1, true, x, x_stride,   \
                        positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, (TA*)q_out,   \
-                       q_stride, (TA*)cache, slots, T, H, G, D, V, page_size, n_pages, err, cv);                   \
+                       q_stride, (TA*)cache, slots, T, H, G, D, V, page_size, n_pages, err, cv, by2);              \
   } while (0)
   if (dtype == SGLC_F32) {
     if (conv) PREP(float, true);
@@ -383,7 +475,7 @@ SGLC_API int sglc_qk_prep_conv(const float* x, long long x_stride, const int* po
                                int dtype, int* err, const float* taps, float* tail, const int* token_req,
                                const int* q_start, const int* state_slots, int K, int n_slots, int own_tail,
                                cudaStream_t stream) {
-  QkConv cv = {taps, tail, token_req, q_start, state_slots, K, n_slots, own_tail};
+  QkConv cv = {taps, tail, token_req, q_start, state_slots, K, n_slots, own_tail, 0};
   return qk_prep_run(x, x_stride, positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, q_out,
                      q_stride, cache, slots, T, H, G, D, V, page_size, n_pages, dtype, err, stream, &cv);
 }

@@ -545,8 +545,12 @@ class RotaryAttention(Part):
                 return self.out.forward(ctx, o, out=out, residual=residual)
         # every other step goes to the general kernel; where every request brings one token, a
         # token's keys are dealt to several blocks and a second launch merges their shares
-        splits = ops.attention_ext_splits(ctx.max_keys, p.get("window"), p.get("chunk")) if ctx.max_q_len == 1 else 1
-        ws = ctx.alloc((T * H * splits * (V + 2),), torch.float32) if splits > 1 else None
+        # (also one share a token, where query heads that share keys gain from staging them once)
+        splits, ws = 1, None
+        if ctx.max_q_len == 1:
+            splits = ops.attention_ext_splits(ctx.max_keys, p.get("window"), p.get("chunk"), T * G)
+            if splits > 1 or 2 <= H // G <= 8:
+                ws = ctx.alloc((T * H * splits * (V + 2),), torch.float32)
         ops.attention_ext(q, cache.tensor, grp.block_table, ctx.token_req, ctx.positions, o, H, G, D, V, grp.page_size,
                           float(p["scale"]), p.get("window"), p.get("chunk"), self.sink, ctx.max_keys,
                           max_q_len=ctx.max_q_len, splits=splits, workspace=ws, gate=gate)

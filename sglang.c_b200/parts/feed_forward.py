@@ -187,18 +187,23 @@ class RoutedExperts(Part):
         from ..csrc import ops
         p = self.params
         T, F, X, top = h.shape[0], p["inner_size"], p["n_experts"], p["top"]
-        z = ctx.alloc((T, self.router.out_size), torch.float32)
-        self.router.forward(ctx, h, out=z)
         n_id = int(p.get("n_identity") or 0)
         dense = ctx.alloc((T, X + n_id), torch.float32)
         passed = ctx.alloc((T,), torch.float32) if n_id else None
         ids = ctx.alloc((T, top), torch.int32)
         wts = ctx.alloc((T, top), torch.float32)
         renorm = bool(p.get("renorm", False))
-        ops.router(ctx.columns(z, 0, X + n_id), self.correction, dense, ids, wts, top, p.get("n_groups", 1), p.get("keep", 1),
+        z = rows = matrix = None
+        if ops.router_product_pays(T, self.router.weight):
+            rows, matrix = h, self.router.weight
+        else:
+            z = ctx.alloc((T, self.router.out_size), torch.float32)
+            self.router.forward(ctx, h, out=z)
+            z = ctx.columns(z, 0, X + n_id)
+        ops.router(z, self.correction, dense, ids, wts, top, p.get("n_groups", 1), p.get("keep", 1),
                    renorm=renorm, weight_scale=float(p.get("weight_scale", 1.0)), score=p.get("score", "sigmoid"),
                    renorm_eps=1e-20 if renorm else 0.0, group_score=p.get("group_score", "top2_sum"), n_pass=n_id,
-                   handed_on=passed)
+                   handed_on=passed, rows=rows, matrix=matrix)
         Fall = X * F + int(p.get("shared_inner_size") or 0)      # the shared expert's columns take weight 1
         gu = ctx.alloc((T, 2 * Fall), self.rt.act_dtype)
         self.gate_up.forward(ctx, h, out=gu)
