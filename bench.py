@@ -907,7 +907,7 @@ def lubavik_step_bytes(cfg, batch, context, prompt_tokens):
 def fupapel_config(base, n_layer):
     """A Fupapel model with the layer sizes of a GPT-2 model: the same width, depth, head size (64) and
     vocabulary.  Layers in fours: chunked attention behind convolutions of four taps (the model's heads
-    over a quarter as many key/value heads, chunks of 320, scaled rotation); latent attention (the model's
+    over a quarter as many key/value heads, chunks of 768, scaled rotation); latent attention (the model's
     heads of 64 plus 32 turned entries over a latent of 96, so a cached row of 128; queries through a
     latent of half the width); chunked attention with gated results (the same heads and chunks); and the
     first kind again with the first layer's keys and values.  Every layer has a mixture of 8 experts of a
@@ -915,7 +915,7 @@ def fupapel_config(base, n_layer):
     E, H, I = base["n_embd"], base["n_head"], base["n_inner"]
     moe = {"kind": "moe", "expert": {"ff": max(64, (I // 6) // 64 * 64)},
            "router": {"experts": 8, "top": 2, "identity": 2, "groups": {"count": 2, "keep": 1}}}
-    chunked = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": 320}}
+    chunked = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": 768}}
     conv = dict(chunked, conv=4, rot={"base": 10000.0, "dims": 64,
                                       "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 256}})
     latent = {"heads": H, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 96, "q_rank": E // 2, "scale": 96 ** -0.5,

@@ -205,6 +205,7 @@ SGLC_API int sglc_latent_rope(const float* qx, long long qx_stride, const float*
 // the thread that reads a channel's tail moves it on; otherwise a launch behind this one does
 // (short_conv.cu: short_conv_tail_kernel), when nobody reads a tail any more.
 constexpr int QK_WARPS = 8;      // (a token's head rows are dealt to the warps: eight keep the rounds few)
+constexpr int QK_MAX_THREADS = 512;      // of a block where the entries lie flat before it
 
 __device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
 __device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) {
@@ -221,18 +222,18 @@ struct QkConv {
 };
 
 template <typename TA, bool CONV>
-__global__ void __launch_bounds__(QK_WARPS * 32)
+__global__ void __launch_bounds__(QK_MAX_THREADS)
 qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __restrict__ positions,
                const double* __restrict__ freq, float mult, int dims, int pairing, int norm_mode, float eps,
                const float* __restrict__ gain_q, const float* __restrict__ gain_k, float v_mult,
                TA* __restrict__ q_out, long long q_stride, TA* __restrict__ cache, const int* __restrict__ slots,
                int T, int H, int G, int D, int V, int page_size, int n_pages, int* err, const QkConv cv, int by2) {
   __shared__ float buf[QK_WARPS][ROT_MAX_DIM];
-  __shared__ float red[2][QK_WARPS];
+  __shared__ float red[2][QK_MAX_THREADS / 32];
   __shared__ float2 turn[ROT_MAX_DIM / 2];     // (cosine, sine) of the token's pairs, made once for all its heads
   extern __shared__ __align__(16) float conv_row[];      // CONV: the token's convolved channels
   pdl_launch_dependents();
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, threads = blockDim.x;
   // (positions and slots are the step's own arrays: no kernel of the step writes them)
   const int pos = positions[t];
   const int slot = G > 0 ? slots[t] : -1;
@@ -240,7 +241,7 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
   const bool page_ok = G > 0 && slot >= 0 && sglc_index_ok(page, n_pages, err);
   const size_t page_elems = (size_t)G * page_size * (D + V);
   const float* xr = x + (size_t)t * x_stride;
-  for (int i = threadIdx.x; i < dims / 2; i += QK_WARPS * 32) {
+  for (int i = threadIdx.x; i < dims / 2; i += threads) {
     double a = (double)pos * freq[i];
     a -= floor(a * 0.15915494309189535) * 6.283185307179586;
     float sn, cs;
@@ -254,7 +255,7 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
     float* tail = cv.tail + (size_t)slot_r * (K - 1) * C;
     pdl_wait();
     if (cv.by4) {
-      for (int ch = threadIdx.x * 4; ch < C; ch += QK_WARPS * 32 * 4) {
+      for (int ch = threadIdx.x * 4; ch < C; ch += threads * 4) {
         float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         for (int j = 0; j < K; j++) {
           const int back = K - 1 - j;          // the input so many tokens ago
@@ -271,7 +272,7 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
         }
       }
     } else {
-      for (int ch = threadIdx.x; ch < C; ch += QK_WARPS * 32) {
+      for (int ch = threadIdx.x; ch < C; ch += threads) {
         float acc = 0.0f;
         for (int j = 0; j < K; j++) {
           const int back = K - 1 - j;
@@ -296,14 +297,25 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
     // one root mean square over all query heads, one over all key heads: every thread sums its
     // share in a fixed order, so a token's bits do not depend on the rest of the step
     float sq = 0.0f, sk = 0.0f;
-    for (int i = threadIdx.x; i < H * D; i += QK_WARPS * 32) sq = fmaf(xr[i], xr[i], sq);
-    for (int i = threadIdx.x; i < G * D; i += QK_WARPS * 32) sk = fmaf(xr[H * D + i], xr[H * D + i], sk);
+    if (by2) {
+      for (int i = threadIdx.x; i < H * D / 2; i += threads) {
+        const float2 v = reinterpret_cast<const float2*>(xr)[i];
+        sq = fmaf(v.x, v.x, fmaf(v.y, v.y, sq));
+      }
+      for (int i = threadIdx.x; i < G * D / 2; i += threads) {
+        const float2 v = reinterpret_cast<const float2*>(xr + H * D)[i];
+        sk = fmaf(v.x, v.x, fmaf(v.y, v.y, sk));
+      }
+    } else {
+      for (int i = threadIdx.x; i < H * D; i += threads) sq = fmaf(xr[i], xr[i], sq);
+      for (int i = threadIdx.x; i < G * D; i += threads) sk = fmaf(xr[H * D + i], xr[H * D + i], sk);
+    }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
     __syncthreads();
     sq = 0.0f; sk = 0.0f;
-    for (int w = 0; w < QK_WARPS; w++) { sq += red[0][w]; sk += red[1][w]; }
+    for (int w = 0; w < threads / 32; w++) { sq += red[0][w]; sk += red[1][w]; }
     inv_all[0] = 1.0f / sqrtf(sq / (float)(H * D) + eps);
     if (G > 0) inv_all[1] = 1.0f / sqrtf(sk / (float)(G * D) + eps);
   }
@@ -314,7 +326,7 @@ qk_prep_kernel(const float* __restrict__ x, long long x_stride, const int* __res
     const int h2 = half / 2, p2 = (D - dims) / 2, n_turn = (H + G) * h2, n_pass = (H + G) * p2;
     TA* qt = q_out + (size_t)t * q_stride;
     TA* kt = G > 0 ? cache + (size_t)page * page_elems + (size_t)off * D : nullptr;
-    for (int unit = threadIdx.x; unit < n_turn + n_pass + G * V / 2; unit += QK_WARPS * 32) {
+    for (int unit = threadIdx.x; unit < n_turn + n_pass + G * V / 2; unit += threads) {
       if (unit >= n_turn + n_pass) {
         const int e = (unit - n_turn - n_pass) * 2, g = e / V, d = e % V;
         if (page_ok) {
@@ -437,11 +449,19 @@ static int qk_prep_run(const float* x, long long x_stride, const int* positions,
   // pairs of entries side by side: even sizes and halves, addresses that allow two floats a load
   const int by2 = pairing == 0 && dims % 4 == 0 && D % 2 == 0 && V % 2 == 0 && x_stride % 2 == 0 && q_stride % 2 == 0 &&
                   (((uintptr_t)x | (uintptr_t)gain_q | (uintptr_t)gain_k | (uintptr_t)q_out | (uintptr_t)cache) & 7) == 0;
+  // In a step of few tokens a block is wide enough for one round over its entries; in a long one the SMs are
+  // full and narrower blocks wait less at their barriers.  (The width decides the order of a token's sums:
+  // it follows from the query heads alone, so a layer with keys and one without give the same queries.)
+  int threads = QK_WARPS * 32;
+  if (T <= 2 * 148 && by2 && (norm_mode == 0 || norm_mode == 3)) {
+    threads = (H * D / 2 + 31) / 32 * 32;
+    threads = threads < 128 ? 128 : threads > QK_MAX_THREADS ? QK_MAX_THREADS : threads;
+  }
 #define PREP(TA, CV)                                                                                               \
   do {                                                                                                             \
     if (smem > 24 * 1024)                                                                                          \
       cudaFuncSetAttribute(qk_prep_kernel<TA, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
-    return sglc_launch(qk_prep_kernel<TA, CV>, dim3(T), dim3(QK_WARPS * 32), smem, stream, 1, true, x, x_stride,   \
+    return sglc_launch(qk_prep_kernel<TA, CV>, dim3(T), dim3(threads), smem,          stream, 1, true, x, x_stride,   \
                        positions, freq, mult, dims, pairing, norm_mode, eps, gain_q, gain_k, v_mult, (TA*)q_out,   \
                        q_stride, (TA*)cache, slots, T, H, G, D, V, page_size, n_pages, err, cv, by2);              \
   } while (0)
