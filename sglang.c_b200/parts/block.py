@@ -115,8 +115,8 @@ class ParallelSublayersBlock(Part):
 
 @register_part("block", "parallel_two_norms")
 class ParallelTwoNormsBlock(Part):
-    """A norm for each of two parallel sublayers: x += mixer(norm1(x)) + ffn(norm2(x)), both of the
-    same x; the feed-forward is there only if the layer has an `ffn`.  With a `shift` sub-part (category
+    """A norm for each of two parallel sublayers: x += mixer(norm1(x)) + ffn(norm2(x)), one x for
+    both; the feed-forward is there only if the layer has an `ffn`.  With a `shift` sub-part (category
     token_mix) what the mixer reads is first mixed with the tokens before.  Both norms (RMS, one eps,
     no biases) and the shift are one launch, so the sublayers' last products may add into the 32-bit
     stream from their epilogues as each ends."""
