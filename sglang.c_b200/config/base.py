@@ -7,6 +7,7 @@ whose absence has a meaning defined by the architecture have defaults.
 """
 import json
 import os
+from dataclasses import dataclass
 
 
 class ConfigError(ValueError):
@@ -99,3 +100,26 @@ def get_str(d, keys, default=_MISSING, choices=None):
     if choices is not None and v not in choices:
         raise ConfigError(f"config.json: key '{k}' is '{v}', known values: {sorted(choices)}")
     return v
+
+
+@dataclass(frozen=True)
+class LayerLoop:
+    """Layers start .. stop-1 run `times` times in a row with the same weights."""
+    start: int
+    stop: int
+    times: int
+
+    @classmethod
+    def read(cls, lp, n_layers):
+        """The value of a model's key 'loop' (None: no layer repeats)."""
+        if lp is None:
+            return None
+        if not isinstance(lp, dict):
+            raise ConfigError("config.json: key 'loop' must be null or an object with 'start', 'stop', 'times'")
+        loop = cls(get_int(lp, "start", minimum=0), get_int(lp, "stop", minimum=1), get_int(lp, "times", minimum=1))
+        if not loop.start < loop.stop <= n_layers:
+            raise ConfigError(f"config.json: loop {loop.start}..{loop.stop} does not lie within the {n_layers} layers")
+        return loop
+
+    def to_dict(self):
+        return {"start": self.start, "stop": self.stop, "times": self.times}

@@ -24,7 +24,7 @@ request's length (positions are computed, not looked up).
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
-from .base import ConfigError, get_float, get_int, get_str
+from .base import ConfigError, LayerLoop, get_float, get_int, get_str
 
 LAYER_TYPES = ("attention", "hgrn2", "latent_attention")
 DEFAULT_MAX_POSITIONS = 1 << 16
@@ -130,16 +130,6 @@ class BuboraxLayer:
 
 
 @dataclass(frozen=True)
-class LayerLoop:
-    start: int
-    stop: int
-    times: int
-
-    def to_dict(self):
-        return {"start": self.start, "stop": self.stop, "times": self.times}
-
-
-@dataclass(frozen=True)
 class BuboraxConfig:
     vocab: int
     width: int
@@ -181,14 +171,7 @@ class BuboraxConfig:
             except ConfigError as e:
                 raise ConfigError(f"{e} (in {where}.mixer)") from None
             layers.append(BuboraxLayer(kind, mixer, ff))
-        loop = None
-        if d.get("loop") is not None:
-            lp = d["loop"]
-            if not isinstance(lp, dict):
-                raise ConfigError("config.json: key 'loop' must be null or an object with 'start', 'stop', 'times'")
-            loop = LayerLoop(get_int(lp, "start", minimum=0), get_int(lp, "stop", minimum=1), get_int(lp, "times", minimum=1))
-            if not loop.start < loop.stop <= len(layers):
-                raise ConfigError(f"config.json: loop {loop.start}..{loop.stop} does not lie within the {len(layers)} layers")
+        loop = LayerLoop.read(d.get("loop"), len(layers))
         return cls(vocab=get_int(d, "vocab", minimum=1), width=width, norm_eps=get_float(norm, "eps", positive=True),
                    norm_groups=groups, residual_mult=get_float(d, "residual_mult", default=1.0), layers=tuple(layers),
                    loop=loop, max_positions=get_int(d, "max_positions", default=DEFAULT_MAX_POSITIONS, minimum=1),

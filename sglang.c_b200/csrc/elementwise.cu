@@ -100,12 +100,23 @@ SGLC_API int sglc_xielu(const void* src, long long src_stride, int src_dtype, vo
 // src holds the F gate columns, then the F up columns.  With `w` (float [rows][F / per]) a block of
 // `per` columns is one expert of a mixture and takes the token's weight for it (zero: not chosen);
 // columns from `n_weighted` on (an expert that every token uses, laid behind the routed ones) take 1.
-// `act` chooses the gate's function (silu, or the tanh form of GELU); `mult` is one more factor of
+// `act` chooses the gate's function (silu, or the tanh form of GELU; or the clamped form, where gate and up
+// are bounded first, g = min(gate, limit), u = clamp(up, -limit, limit), and the result is
+// g sigmoid(slope g) (u + 1)); `mult` is one more factor of
 // every result (a layer's residual multiplier, taken in 32-bit ahead of the rounding).
 // `pass` (rows of E, optional): the same launch also forms x[r][c] = w_pass[r] * h[r][c] (added to x
 // with `add`): the experts of a mixture that hand their input on as it is, summed straight into the
 // 32-bit rows that the down product adds to.
-enum { GA_SILU = 0, GA_GELU_TANH = 1 };
+enum { GA_SILU = 0, GA_GELU_TANH = 1, GA_CLAMPED = 2 };
+struct GateFn { int act; float slope, limit; };
+__device__ __forceinline__ float gate_up(const GateFn& f, float g, float u) {
+  if (f.act == GA_CLAMPED) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit);
+    return g / (1.0f + expf(-f.slope * g)) * (u + 1.0f);
+  }
+  return (f.act == GA_GELU_TANH ? gelu_tanh_f32(g) : g / (1.0f + expf(-g))) * u;
+}
 struct PassRows {
   const void* h; long long h_stride;      // in the activation precision (null: none)
   const float* w;                         // [rows]
@@ -155,7 +166,7 @@ __device__ __forceinline__ void pass_rows(const PassRows& p, int rows) {
 template <typename TI, typename TO>
 __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_stride, TO* __restrict__ dst,
                                  long long dst_stride, int rows, int F, const float* __restrict__ w,
-                                 long long w_stride, int per, int act, float mult, int n_weighted,
+                                 long long w_stride, int per, const GateFn fn, float mult, int n_weighted,
                                  const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
@@ -169,7 +180,7 @@ __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_strid
     float out = 0.0f;
     if (wt != 0.0f) {
       const float g = to_f32(src[r * src_stride + c]), u = to_f32(src[r * src_stride + F + c]);
-      out = (act == GA_GELU_TANH ? gelu_tanh_f32(g) : g / (1.0f + expf(-g))) * u * (wt * mult);
+      out = gate_up(fn, g, u) * (wt * mult);
     }
     dst[r * dst_stride + c] = from_f32<TO>(out);
   }
@@ -179,7 +190,7 @@ __global__ void gated_act_kernel(const TI* __restrict__ src, long long src_strid
 // multiples of 8, rows 16-byte aligned
 __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, long long src_stride,
                                       __nv_bfloat16* __restrict__ dst, long long dst_stride, int rows, int F,
-                                      const float* __restrict__ w, long long w_stride, int per, int act, float mult,
+                                      const float* __restrict__ w, long long w_stride, int per, const GateFn fn, float mult,
                                       int n_weighted, const PassRows pass) {
   pdl_launch_dependents();
   pdl_wait();
@@ -201,10 +212,7 @@ __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, lon
 #pragma unroll
       for (int k = 0; k < 4; k++) {
         const float2 g = __bfloat1622float2(gp[k]), u = __bfloat1622float2(up[k]);
-        if (act == GA_GELU_TANH)
-          op[k] = __floats2bfloat162_rn(gelu_tanh_f32(g.x) * u.x * wt, gelu_tanh_f32(g.y) * u.y * wt);
-        else
-          op[k] = __floats2bfloat162_rn(g.x / (1.0f + expf(-g.x)) * u.x * wt, g.y / (1.0f + expf(-g.y)) * u.y * wt);
+        op[k] = __floats2bfloat162_rn(gate_up(fn, g.x, u.x) * wt, gate_up(fn, g.y, u.y) * wt);
       }
     }
     *reinterpret_cast<uint4*>(dst + r * dst_stride + c) = o;
@@ -214,9 +222,9 @@ __global__ void gated_act_vec8_kernel(const __nv_bfloat16* __restrict__ src, lon
 // n_weighted: the first so many columns (a multiple of `per`) take weights, the rest take 1
 static int gated_act_run(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,
                          int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
-                         int act, float mult, int n_weighted, PassRows pass, cudaStream_t stream) {
+                         GateFn fn, float mult, int n_weighted, PassRows pass, cudaStream_t stream) {
   if (rows <= 0 || F <= 0) return SGLC_OK;
-  if (act != GA_SILU && act != GA_GELU_TANH) return SGLC_ERR_ARGUMENT;
+  if (fn.act < GA_SILU || fn.act > GA_CLAMPED || (fn.act == GA_CLAMPED && !(fn.limit > 0.0f))) return SGLC_ERR_ARGUMENT;
   if (w && (per <= 0 || n_weighted < 0 || n_weighted > F || n_weighted % per != 0)) return SGLC_ERR_ARGUMENT;
   const long long total = (long long)rows * F;
   int blocks = (int)((total + 255) / 256);
@@ -236,12 +244,12 @@ static int gated_act_run(const void* src, long long src_stride, int src_dtype, v
     if (b8 > 148 * 16) b8 = 148 * 16;
     pass.first_block = b8;
     return sglc_launch(gated_act_vec8_kernel, dim3(b8 + more), dim3(256), 0, stream, 1, true, (const __nv_bfloat16*)src,
-                       src_stride, (__nv_bfloat16*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult,
+                       src_stride, (__nv_bfloat16*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, fn, mult,
                        n_weighted, pass);
   }
 #define LAUNCH(TI, TO)                                                                                  \
   return sglc_launch(gated_act_kernel<TI, TO>, dim3(blocks + more), dim3(256), 0, stream, 1, true, (const TI*)src, \
-                     src_stride, (TO*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, act, mult, n_weighted, pass)
+                     src_stride, (TO*)dst, dst_stride, rows, F, w, w_stride, per > 0 ? per : 1, fn, mult, n_weighted, pass)
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_F32) LAUNCH(float, float);
   if (src_dtype == SGLC_F32 && dst_dtype == SGLC_BF16) LAUNCH(float, __nv_bfloat16);
   if (src_dtype == SGLC_BF16 && dst_dtype == SGLC_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
@@ -253,8 +261,17 @@ SGLC_API int sglc_gated_act_part(const void* src, long long src_stride, int src_
                                  int dst_dtype, int rows, int F, const float* w, long long w_stride, int per,
                                  int act, float mult, int n_weighted, cudaStream_t stream) {
   PassRows none = {};
-  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per, act, mult,
-                       n_weighted, none, stream);
+  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per,
+                       GateFn{act, 0.0f, 0.0f}, mult, n_weighted, none, stream);
+}
+
+// The clamped form: dst[r][j] = g sigmoid(slope g) (u + 1) * mult, g = min(gate, limit), u = clamp(up, +-limit).
+SGLC_API int sglc_gated_act_clamped(const void* src, long long src_stride, int src_dtype, void* dst,
+                                    long long dst_stride, int dst_dtype, int rows, int F, float slope, float limit,
+                                    float mult, cudaStream_t stream) {
+  PassRows none = {};
+  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, nullptr, 0, 0,
+                       GateFn{GA_CLAMPED, slope, limit}, mult, F, none, stream);
 }
 
 // With rows handed on: x[r][c] (+)= w_pass[r] * h[r][c], c < E; h in dst's precision, x 32-bit.
@@ -265,8 +282,8 @@ SGLC_API int sglc_gated_act_pass(const void* src, long long src_stride, int src_
                                  cudaStream_t stream) {
   if (!h || !w_pass || !x || E <= 0) return SGLC_ERR_ARGUMENT;
   PassRows pass = {h, h_stride, w_pass, x, x_stride, E, add, 0, 0};
-  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per, act, mult,
-                       n_weighted, pass, stream);
+  return gated_act_run(src, src_stride, src_dtype, dst, dst_stride, dst_dtype, rows, F, w, w_stride, per,
+                       GateFn{act, 0.0f, 0.0f}, mult, n_weighted, pass, stream);
 }
 
 SGLC_API int sglc_gated_act_ext(const void* src, long long src_stride, int src_dtype, void* dst, long long dst_stride,

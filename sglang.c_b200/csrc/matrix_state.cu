@@ -16,7 +16,9 @@
 //       S <- g_t S + b_t k_t v_t^T                     o_t = S^T q_t
 //     with `ones_col` the state has one more column than v has entries, whose "value" is 1 for every
 //     token: it carries sum_t b_t k_t under the same decay (a normaliser), and its read-out n_t . q_t
-//     leaves in the last column of the head's output.
+//     leaves in the last column of the head's output.  With `skip` (a number per head) the token's own
+//     value joins the result: o_t = S^T q_t + skip_h v_t  (a selective state space, Mamba-2: b_t is the step
+//     size, k_t and q_t are what it calls B and C).
 // in this order: the read-out sees the current token's write.
 //
 // Column j of S needs nothing of the other columns: S^T k, the update and S^T q are, per column,
@@ -50,6 +52,7 @@ struct MsArgs {
   float inv_tau;                          // row-decay form: a = exp(log sigmoid(z) * inv_tau)
   float q_scale;                          // a factor of q
   int ones_col;                           // gated form: the state's last column takes the value 1
+  const float* skip;                      // gated form: null, or [H] factors of the token's own value in its result
   const float* head_decay;                // decay form: [H]
   const float* lower;                     // row-gated form: [H*D] lower bounds of the forget gates
   float* out; long long out_stride;       // [T][H*V]
@@ -100,6 +103,7 @@ matrix_state_kernel(MsArgs p) {
     S[e] = (on && i < p.D) ? sp[(size_t)i * p.V + col] : 0.0f;
   }
   const float hd = MODE == MS_DECAY ? p.head_decay[h] : 0.0f;
+  const float skip = (MODE == MS_GATED && p.skip) ? p.skip[h] : 0.0f;
   float* out_row = p.out + (size_t)h * p.V + col;
   float rk[NK], rq[NK], rv[NV], rg[NG], ra[ROWA ? NK : 1];
   const int v_in = p.ones_col ? p.V - 1 : p.V;          // entries a head of v has
@@ -269,6 +273,7 @@ matrix_state_kernel(MsArgs p) {
     auto finish = [&](int b, float o) {
 #pragma unroll
       for (int m = 1; m < L; m <<= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
+      if (MODE == MS_GATED) o = fmaf(skip, vs[buf][b * COLS + lcol], o);
       if (on && sub == 0)
         asm volatile("st.global.f32 [%0], %1;" ::"l"(out_row + (size_t)(tb + b) * p.out_stride), "f"(o));
     };
@@ -327,12 +332,13 @@ SGLC_API void sglc_matrix_state_set_per(int per) { g_ms_per = per; }
 // mode 3: row-decay form (row_z [T][G*D] the decays' pre-activations, inv_tau = 1 / tau).
 // mode 4: gated form (gates [T][2H]: input weight, decay); ones_col: the state has V columns of which
 // the last takes the value 1 (v then has heads of V - 1 entries; out still has heads of V).
+// skip (mode 4): null, or [H] factors of the token's own value, added to its result.
 // q_scale: a factor of q (1 for none).
 SGLC_API int sglc_matrix_state_gen(int mode, const float* q, long long q_stride, const float* k, long long k_stride,
                                    const float* v, long long v_stride, const float* gates, long long gates_stride,
                                    const float* head_decay, const float* lower, const float* row_z,
-                                   long long row_z_stride, float inv_tau, float q_scale, int ones_col, float* out,
-                                   long long out_stride, float* state, int n_slots, const int* q_start,
+                                   long long row_z_stride, float inv_tau, float q_scale, int ones_col,
+                                   const float* skip, float* out, long long out_stride, float* state, int n_slots, const int* q_start,
                                    const int* state_slots, int R, int H, int G, int D, int V, int silu_in, int* err,
                                    cudaStream_t stream) {
   if (R <= 0) return SGLC_OK;
@@ -345,6 +351,8 @@ SGLC_API int sglc_matrix_state_gen(int mode, const float* q, long long q_stride,
   p.R = R; p.H = H; p.G = G; p.D = D; p.V = V; p.n_slots = n_slots; p.silu_in = silu_in; p.err = err;
   p.row_z = row_z; p.row_z_stride = row_z_stride; p.inv_tau = inv_tau; p.q_scale = q_scale;
   p.ones_col = mode == MS_GATED && ones_col ? 1 : 0;
+  p.skip = skip;
+  if (skip && mode != MS_GATED) return SGLC_ERR_ARGUMENT;
   if (p.ones_col && V < 2) return SGLC_ERR_ARGUMENT;
   // Entries a lane keeps: 8 for key sizes of 33..64 while the warps still find a scheduler each (two
   // on each of the 148 x 4); else 16.
@@ -397,7 +405,7 @@ SGLC_API int sglc_matrix_state_ext(int mode, const float* q, long long q_stride,
                                    int G, int D, int V, int silu_in, int* err, cudaStream_t stream) {
   if (mode > MS_ROWGATE) return SGLC_ERR_ARGUMENT;
   return sglc_matrix_state_gen(mode, q, q_stride, k, k_stride, v, v_stride, gates, gates_stride, head_decay, lower,
-                               nullptr, 0, 0.0f, 1.0f, 0, out, out_stride, state, n_slots, q_start, state_slots, R, H, G,
+                               nullptr, 0, 0.0f, 1.0f, 0, nullptr, out, out_stride, state, n_slots, q_start, state_slots, R, H, G,
                                D, V, silu_in, err, stream);
 }
 

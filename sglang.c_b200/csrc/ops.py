@@ -854,6 +854,46 @@ def depth_mix(x, hist, n_terms, weights):
     _check(lib, code, "depth_mix")
 
 
+STREAMS_MAX = 32
+
+
+def stream_step(src, h, w_in, gain=None, eps=0.0, write=None, rows=None):
+    """One launch between two sublayers of a model with S residual streams (stream_step.cu).
+    src: float32 [T, S, E], the streams (a stride of 0 between streams: S copies of one row).
+    write = (y, w_out, w_mix, dst): first X_t <- sum_s w_mix[s, t] X_s + w_out[t] y, y float32 [T, E], the
+    new streams into dst [T, S, E] (may be src; None: they are only read from).  Then
+    h = sum_s w_in[s] X_s, RMS-normed with `gain` (float32 [E]) and eps if a gain is given; h [T, E]
+    float32 or bfloat16.  rows (int32): only these rows, read and written at their places."""
+    y, w_out, w_mix, dst = write if write is not None else (None, None, None, None)
+    _need_cuda(src, h, w_in, gain, y, w_out, w_mix, dst, rows)
+    T, S, E = src.shape
+    if src.dtype != torch.float32 or src.stride(2) != 1 or h.stride(1) != 1 or tuple(h.shape) != (T, E):
+        raise KernelError("stream_step: src float32 [T, S, E], h [T, E]")
+    if S > STREAMS_MAX:
+        raise KernelError(f"stream_step: {S} streams are beyond the kernel's {STREAMS_MAX}")
+    for v, n, nm in ((w_in, S, "w_in"), (gain, E, "gain"), (w_out, S, "w_out"), (w_mix, S * S, "w_mix")):
+        if v is not None and (v.dtype != torch.float32 or v.numel() != n or not v.is_contiguous()):
+            raise KernelError(f"stream_step: {nm} is a contiguous float32 tensor of {n}")
+    if y is not None:
+        _f32_rows(y, "stream_step: y", E)
+        if y.shape[0] < T:
+            raise KernelError("stream_step: y has a row for every token")
+    if dst is not None and (dst.dtype != torch.float32 or dst.stride(2) != 1 or tuple(dst.shape) != (T, S, E)):
+        raise KernelError("stream_step: dst float32 [T, S, E]")
+    n = T
+    if rows is not None:
+        _i32(rows, "rows")
+        n = rows.numel()
+    lib = build.load("stream_step")
+    code = lib.sglc_stream_step(
+        _ptr(src), ctypes.c_longlong(src.stride(0)), ctypes.c_longlong(src.stride(1)), _ptr(dst),
+        ctypes.c_longlong(dst.stride(0) if dst is not None else 0), ctypes.c_longlong(dst.stride(1) if dst is not None else 0),
+        _ptr(y), ctypes.c_longlong(y.stride(0) if y is not None else 0), _ptr(w_out), _ptr(w_mix), _ptr(w_in), _ptr(gain),
+        ctypes.c_float(eps), _ptr(h), ctypes.c_longlong(h.stride(0)), _dt(h, "stream_step output"), _ptr(rows), int(n), T,
+        S, E, _ptr(tc_error_flag(src.device)), _stream())
+    _check(lib, code, f"stream_step ({S} streams, width {E})")
+
+
 def xielu(src, dst, ap, an):
     """dst = xIELU(src): ap*x^2 + x/2 for x > 0, an*(exp(x)-1-x) + x/2 otherwise."""
     _need_cuda(src, dst)
@@ -930,12 +970,46 @@ def short_conv(x, taps, tail, y, token_req, q_start, state_slots, n_requests, se
     _check(lib, code, f"short_conv (channels {C}, taps {K})", n_kernels=2 if K > 1 and T != int(n_requests) else 1)
 
 
+def conv_silu(x, taps, bias, tail, y, token_req, q_start, state_slots, n_requests, gates=None):
+    """y = silu(bias + causal convolution over time of x's first C columns) (short_conv.cu:
+    conv_silu_kernel).  x: float32 [T, >= C]; taps: float32 [K, C] (the last row is the current token's);
+    bias: float32 [C]; tail: float32 [n_slots, K-1, C], a request's last K-1 inputs, read and moved on
+    in place; y: float32 [T, C].  gates = (heads, column, A_log, dt_bias, out [T, 2*heads]): per head
+    dt = softplus(x_column + dt_bias) and exp(-exp(A_log) dt), from one more column block of x."""
+    _need_cuda(x, taps, bias, tail, y, token_req, q_start, state_slots)
+    T = y.shape[0]
+    K, C = taps.shape
+    _f32_rows(x, "conv_silu: x")
+    _f32_rows(y, "conv_silu: y", C)
+    if taps.dtype != torch.float32 or not taps.is_contiguous() or x.shape[0] < T or x.shape[1] < C \
+            or bias.dtype != torch.float32 or bias.numel() != C or not bias.is_contiguous():
+        raise KernelError("conv_silu: taps float32 [K, C], bias float32 [C]; x has at least C columns")
+    if tail.dtype != torch.float32 or not tail.is_contiguous() or tuple(tail.shape[1:]) != (max(K - 1, 0), C):
+        raise KernelError(f"conv_silu: the tail is float32 [n_slots, {K - 1}, {C}]")
+    for t, nm in ((token_req, "token_req"), (q_start, "q_start"), (state_slots, "state_slots")):
+        _i32(t, nm)
+    gh, col, a_log, dt_bias, gout = gates if gates is not None else (0, 0, None, None, None)
+    if gates is not None:
+        _need_cuda(a_log, dt_bias, gout)
+        _f32_rows(gout, "conv_silu: gates", 2 * gh)
+        if a_log.dtype != torch.float32 or dt_bias.dtype != torch.float32 or a_log.numel() != gh \
+                or dt_bias.numel() != gh or x.shape[1] < col + gh or gout.shape[0] < T:
+            raise KernelError("conv_silu: A_log and dt_bias are float32 [heads]; x holds the gates' columns")
+    lib = build.load("short_conv")
+    code = lib.sglc_conv_silu(_ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(taps), _ptr(bias), _ptr(tail), _ptr(y),
+                              ctypes.c_longlong(y.stride(0)), _ptr(token_req), _ptr(q_start), _ptr(state_slots), T,
+                              int(n_requests), C, K, tail.shape[0], int(gh), int(col), _ptr(a_log), _ptr(dt_bias),
+                              _ptr(gout), ctypes.c_longlong(gout.stride(0) if gout is not None else 0),
+                              _ptr(tc_error_flag(x.device)), _stream())
+    _check(lib, code, f"conv_silu (channels {C}, taps {K})")
+
+
 MATRIX_STATE_MAX_DIM = 256
 
 
 def matrix_state(mode, q, k, v, out, state, q_start, state_slots, n_requests, n_heads, n_qk_heads, dim, v_dim,
                  gates=None, head_decay=None, silu_in=False, lower=None, row_z=None, tau=1.0, q_scale=1.0,
-                 ones_col=False):
+                 ones_col=False, skip=None):
     """A recurrence with a matrix state per head over the step's tokens (see matrix_state.cu).
     mode "decay": S <- d_h S + k v^T (head_decay float32 [H]); mode "delta": the gated delta rule
     (gates float32 [T, 2H]: beta, then decay); mode "row_gate": S <- diag(f) S + (1 - f) v^T with
@@ -944,7 +1018,8 @@ def matrix_state(mode, q, k, v, out, state, q_start, state_slots, n_requests, n_
     a = sigmoid(row_z)^(1/tau) per head and row (row_z float32 [T, n_qk_heads*dim]); mode "gated":
     S <- g S + b k v^T (gates float32 [T, 2H]: b, then g); with ones_col the state (and out) have
     v_dim columns a head of which the last takes the value 1 for every token, and v has heads of
-    v_dim - 1.  q_scale multiplies q.  o = S^T q after the token's write.  q, k: float32
+    v_dim - 1, or with skip (float32 [H]) o = S^T q + skip_h v.  q_scale multiplies q.  o = S^T q after the
+    token's write.  q, k: float32
     [T, n_qk_heads*dim]; v: float32 [T, n_heads*v_dim]; out float32 [T, n_heads*v_dim]; state float32
     [n_slots, n_heads, dim, v_dim], read and written in place for the requests' slots."""
     _need_cuda(q, k, v, out, state, q_start, state_slots, gates, head_decay, lower)
@@ -962,6 +1037,10 @@ def matrix_state(mode, q, k, v, out, state, q_start, state_slots, n_requests, n_
     m = {"decay": 0, "delta": 1, "row_gate": 2, "row_decay": 3, "gated": 4}[mode]
     if ones_col and m != 4:
         raise KernelError("matrix_state: the column of ones goes with the gated form")
+    if skip is not None:
+        _need_cuda(skip)
+        if m != 4 or ones_col or skip.dtype != torch.float32 or skip.numel() != n_heads or not skip.is_contiguous():
+            raise KernelError("matrix_state: skip is a float32 factor per head of the gated form without a column of ones")
     if m == 3:
         if row_z is None:
             raise KernelError("matrix_state: the row-decay form takes the decays' pre-activations")
@@ -983,7 +1062,7 @@ def matrix_state(mode, q, k, v, out, state, q_start, state_slots, n_requests, n_
                                  ctypes.c_longlong(gates.stride(0) if gates is not None else 0), _ptr(head_decay),
                                  _ptr(lower), _ptr(row_z), ctypes.c_longlong(row_z.stride(0) if row_z is not None else 0),
                                  ctypes.c_float(1.0 / float(tau)), ctypes.c_float(q_scale), 1 if ones_col else 0,
-                                 _ptr(out), ctypes.c_longlong(out.stride(0)), _ptr(state), state.shape[0],
+                                 _ptr(skip), _ptr(out), ctypes.c_longlong(out.stride(0)), _ptr(state), state.shape[0],
                                  _ptr(q_start), _ptr(state_slots), int(n_requests), int(n_heads), int(n_qk_heads),
                                  int(dim), int(v_dim), 1 if silu_in else 0, _ptr(tc_error_flag(q.device)), _stream())
     _check(lib, code, f"matrix_state ({mode}, {dim} x {v_dim})")
@@ -1022,6 +1101,25 @@ def gated_norm(o, gate, gain, y, groups, width, eps, act, o_pitch=None, m_run=No
                                    1 if (gain.numel() == groups * width and groups > 1) else 0, _ptr(m_run),
                                    ctypes.c_longlong(m_run.stride(0) if m_run is not None else 0), _stream())
     _check(lib, code, f"gated_norm (width {width})")
+
+
+def gate_then_norm(o, gate, gain, y, groups, width, eps, act):
+    """y = x / sqrt(mean(x^2) + eps) * gain with x = o * act(gate), per part of `width` columns (a token
+    has `groups` of them side by side; gain float32 [groups*width]); act "silu" or "sigmoid".  o, gate:
+    float32 [T, groups*width]; y: float32 or bfloat16."""
+    _need_cuda(o, gate, gain, y)
+    T = y.shape[0]
+    _f32_rows(o, "gate_then_norm: o", groups * width)
+    _f32_rows(gate, "gate_then_norm: gate", groups * width)
+    if gain.dtype != torch.float32 or gain.numel() != groups * width or not gain.is_contiguous():
+        raise KernelError("gate_then_norm: the gain is a float32 vector of the whole row")
+    if tuple(y.shape) != (T, groups * width) or y.stride(1) != 1 or o.shape[0] < T or gate.shape[0] < T:
+        raise KernelError("gate_then_norm: y is [T, groups*width]")
+    lib = build.load("gated_norm")
+    code = lib.sglc_gate_then_norm(_ptr(o), ctypes.c_longlong(o.stride(0)), _ptr(gate), ctypes.c_longlong(gate.stride(0)),
+                                   _ptr(gain), _ptr(y), ctypes.c_longlong(y.stride(0)), _dt(y, "gate_then_norm output"),
+                                   T, int(groups), int(width), ctypes.c_float(eps), {"silu": 0, "sigmoid": 1}[act], _stream())
+    _check(lib, code, f"gate_then_norm (width {width})")
 
 
 def rotary_kv(x, positions, freq, mult, dims, norm_eps, q_out, cache, slots, n_heads, n_kv_heads, dim, v_dim,
@@ -1237,13 +1335,15 @@ def attention_ext(q, cache, block_table, token_req, positions, out, n_heads, n_k
     _check(lib, code, f"attention_ext (head {dim}/{v_dim}, up to {max_keys} keys)")
 
 
-GATE_ACTS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
 
 
-def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=None, handed_on=None):
+def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=None, handed_on=None, slope=None,
+              limit=None):
     """dst[r, j] = act(src[r, j]) * src[r, F + j] (* weights[r, j // per]) * mult; src [rows, 2F] holds
     the gate columns, then the up columns; weights: float32 [rows, F // per] or None; act "silu" or
-    "gelu_tanh"; mult: one more factor of every result, taken in 32-bit.  n_weighted: only the
+    "gelu_tanh", or "clamped" (dst = g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = up held within
+    +-limit; without weights); mult: one more factor of every result, taken in 32-bit.  n_weighted: only the
     first so many columns (a multiple of per) take weights, [rows, n_weighted // per]; the rest take 1.
     handed_on = (h, w, x, add): the same launch forms x[r, :] = w[r] * h[r, :] (added to x if `add`);
     h [rows, E] in dst's dtype, w float32 [rows], x float32 [rows, E]."""
@@ -1259,6 +1359,15 @@ def gated_act(src, dst, weights=None, per=0, act="silu", mult=1.0, n_weighted=No
     else:
         nw = F
     lib = build.load("elementwise")
+    if act == "clamped":
+        if weights is not None or handed_on is not None or slope is None or not (limit or 0) > 0:
+            raise KernelError("gated_act: the clamped form takes slope and limit > 0, no weights, nothing handed on")
+        code = lib.sglc_gated_act_clamped(
+            _ptr(src), ctypes.c_longlong(src.stride(0)), _dt(src, "gated_act source"), _ptr(dst),
+            ctypes.c_longlong(dst.stride(0)), _dt(dst, "gated_act destination"), rows, F, ctypes.c_float(slope),
+            ctypes.c_float(limit), ctypes.c_float(mult), _stream())
+        _check(lib, code, "gated_act")
+        return
     if handed_on is not None:
         h, w, x, add = handed_on
         _need_cuda(h, w, x)

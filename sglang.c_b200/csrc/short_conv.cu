@@ -13,6 +13,9 @@
 //
 // The same launch makes the per-head gates of a gated delta rule from two more columns blocks of x:
 //   beta = sigmoid(x_b),   decay = exp(-exp(A_log) * softplus(x_a + dt_bias)).
+//
+// A second form (conv_silu_kernel) has a bias per channel and no head rows, and makes the gates of a
+// selective state space from one more column block: dt = softplus(x_dt + dt_bias) and exp(-exp(A_log) dt).
 #include "common.cuh"
 
 SGLC_DEFINE_ERROR_STRING()
@@ -183,4 +186,150 @@ SGLC_API int sglc_short_conv_tail(const float* x, long long x_stride, float* tai
   p.x = x; p.x_stride = x_stride; p.tail = tail; p.q_start = q_start; p.state_slots = state_slots;
   p.R = R; p.C = C; p.K = K; p.n_slots = n_slots; p.err = err;
   return sglc_launch(short_conv_tail_kernel, dim3(R, (C + 127) / 128), dim3(128), 0, stream, 1, true, p);
+}
+
+// y_t[ch] = silu(bias[ch] + sum_j taps[j][ch] x_{t-(K-1)+j}[ch]): a thread takes CW neighbouring channels of
+// `per` consecutive tokens of the step and moves a window over them.  Tails in the same launch: the
+// tokens that look back before their portion, its first K-1, all belong to the thread that meets the portion's
+// first token (others pass over them), so a channel's tail has one reader, which then moves it on.
+// The last row of blocks makes the gates.
+struct ConvSiluArgs {
+  const float* x; long long x_stride;       // [T][x_stride], the channels are its first C columns
+  const float* taps; const float* bias;     // [K][C], [C]
+  float* tail;                              // [n_slots][K-1][C]
+  float* y; long long y_stride;             // [T][C]
+  const int* token_req; const int* q_start; const int* state_slots;
+  int T, C, K, n_slots, per;
+  int heads, dt_col;                        // heads = 0: no gates
+  const float* A_log; const float* dt_bias;
+  float* gates; long long gates_stride;     // [T][2 heads]: dt, then the decay
+  int* err;
+};
+
+template <int CW> struct ConvVec;
+template <> struct ConvVec<1> {
+  float v;
+  __device__ static ConvVec load(const float* p) { return {*p}; }
+  __device__ void store(float* p) const { *p = v; }
+  __device__ void fma(const ConvVec& a, const ConvVec& b) { v = fmaf(a.v, b.v, v); }
+  __device__ ConvVec silu() const { return {silu_f32(v)}; }
+};
+template <> struct ConvVec<4> {
+  float4 v;
+  __device__ static ConvVec load(const float* p) { return {*reinterpret_cast<const float4*>(p)}; }
+  __device__ void store(float* p) const { *reinterpret_cast<float4*>(p) = v; }
+  __device__ void fma(const ConvVec& a, const ConvVec& b) {
+    v.x = fmaf(a.v.x, b.v.x, v.x); v.y = fmaf(a.v.y, b.v.y, v.y);
+    v.z = fmaf(a.v.z, b.v.z, v.z); v.w = fmaf(a.v.w, b.v.w, v.w);
+  }
+  __device__ ConvVec silu() const { return {make_float4(silu_f32(v.x), silu_f32(v.y), silu_f32(v.z), silu_f32(v.w))}; }
+};
+
+// KT: the taps as a constant (the window then stays in registers), or 0: any number, inputs read again.
+template <int CW, int KT>
+__global__ void __launch_bounds__(128)
+conv_silu_kernel(const ConvSiluArgs p) {
+  using V = ConvVec<CW>;
+  pdl_launch_dependents();
+  const int ta = blockIdx.x * p.per, tb = min(ta + p.per, p.T);
+  if (p.heads && blockIdx.y == gridDim.y - 1) {
+    pdl_wait();
+    for (int i = threadIdx.x; i < (tb - ta) * p.heads; i += blockDim.x) {
+      const int t = ta + i / p.heads, h = i % p.heads;
+      const float dt = softplus_f32(p.x[(size_t)t * p.x_stride + p.dt_col + h] + p.dt_bias[h]);
+      p.gates[(size_t)t * p.gates_stride + h] = dt;
+      p.gates[(size_t)t * p.gates_stride + p.heads + h] = expf(-expf(p.A_log[h]) * dt);
+    }
+    return;
+  }
+  const int ch = (blockIdx.y * 128 + threadIdx.x) * CW;
+  if (ch >= p.C) return;
+  const int K = KT ? KT : p.K;
+  V w[KT ? KT : 1], win[KT > 1 ? KT - 1 : 1];
+  if constexpr (KT > 0) {
+#pragma unroll
+    for (int j = 0; j < KT; j++) w[j] = V::load(p.taps + (size_t)j * p.C + ch);
+  }
+  const V b = V::load(p.bias + ch);
+  const float* x = p.x + ch;
+  pdl_wait();
+  bool have = false;                         // the window holds the K-1 inputs ahead of token t
+  for (int t = ta; t < tb; t++) {
+    const int r = p.token_req[t];
+    const int q0 = p.q_start[r], i = t - q0;
+    if (i < K - 1) {
+      have = false;
+      if (i > 0) continue;                   // (done with the portion's first token)
+      const int n = p.q_start[r + 1] - q0;
+      const int slot = p.state_slots[r];
+      if (!sglc_index_ok(slot, p.n_slots, p.err)) continue;
+      float* tail = p.tail + (size_t)slot * (K - 1) * p.C + ch;
+      for (int e = 0; e < min(n, K - 1); e++) {
+        V a = b;
+        for (int j = 0; j < K; j++) {
+          const int src = e - (K - 1) + j;
+          a.fma(V::load(p.taps + (size_t)j * p.C + ch),
+                V::load(src >= 0 ? x + (size_t)(q0 + src) * p.x_stride : tail + (size_t)(K - 1 + src) * p.C));
+        }
+        a.silu().store(p.y + (size_t)(q0 + e) * p.y_stride + ch);
+      }
+      for (int m = 0; m < K - 1; m++) {      // ascending: an old entry is read before its place is written
+        const int src = n - (K - 1) + m;
+        V::load(src >= 0 ? x + (size_t)(q0 + src) * p.x_stride : tail + (size_t)(m + n) * p.C).store(tail + (size_t)m * p.C);
+      }
+      continue;
+    }
+    V a = b;
+    if constexpr (KT > 0) {
+      if (!have) {
+#pragma unroll
+        for (int j = 0; j < KT - 1; j++) win[j] = V::load(x + (size_t)(t - (KT - 1) + j) * p.x_stride);
+        have = true;
+      }
+      const V now = V::load(x + (size_t)t * p.x_stride);
+#pragma unroll
+      for (int j = 0; j < KT - 1; j++) a.fma(w[j], win[j]);
+      a.fma(w[KT - 1], now);
+#pragma unroll
+      for (int j = 0; j + 1 < KT - 1; j++) win[j] = win[j + 1];
+      if constexpr (KT > 1) win[KT - 2] = now;
+    } else {
+      for (int j = 0; j < K; j++)
+        a.fma(V::load(p.taps + (size_t)j * p.C + ch), V::load(x + (size_t)(t - (K - 1) + j) * p.x_stride));
+    }
+    a.silu().store(p.y + (size_t)t * p.y_stride + ch);
+  }
+}
+
+// heads > 0: gates from x's columns dt_col .. dt_col + heads - 1 (counted from x's first channel).
+SGLC_API int sglc_conv_silu(const float* x, long long x_stride, const float* taps, const float* bias, float* tail,
+                            float* y, long long y_stride, const int* token_req, const int* q_start,
+                            const int* state_slots, int T, int R, int C, int K, int n_slots, int heads, int dt_col,
+                            const float* A_log, const float* dt_bias, float* gates, long long gates_stride, int* err,
+                            cudaStream_t stream) {
+  if (T <= 0 || R <= 0) return SGLC_OK;
+  if (C <= 0 || K < 1 || (heads > 0 && (!A_log || !dt_bias || !gates)) || heads < 0) return SGLC_ERR_ARGUMENT;
+  if (K > CONV_MAX_TAPS) return SGLC_ERR_UNSUPPORTED;
+  ConvSiluArgs p = {x, x_stride, taps, bias, tail, y, y_stride, token_req, q_start, state_slots, T, C, K, n_slots, 1,
+                    heads, dt_col, A_log, dt_bias, gates, gates_stride, err};
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = C % 4 == 0 && x_stride % 4 == 0 && y_stride % 4 == 0 && al(x) && al(taps) && al(bias) && al(tail) && al(y);
+  const int cb = (C + (vec ? 512 : 128) - 1) / (vec ? 512 : 128);
+  if (cb + 1 > 65535) return SGLC_ERR_UNSUPPORTED;
+  // tokens a thread: as many as still leave every SM several blocks, up to 8
+  while (p.per < 8 && (long long)((T + 2 * p.per - 1) / (2 * p.per)) * cb >= 148LL * 4) p.per *= 2;
+  const dim3 grid((T + p.per - 1) / p.per, cb + (heads > 0 ? 1 : 0));
+#define GO(CW, KT) return sglc_launch(conv_silu_kernel<CW, KT>, grid, dim3(128), 0, stream, 1, true, p)
+#define PICK(CW)        \
+  switch (K) {          \
+    case 1: GO(CW, 1);  \
+    case 2: GO(CW, 2);  \
+    case 3: GO(CW, 3);  \
+    case 4: GO(CW, 4);  \
+    default: GO(CW, 0); \
+  }
+  if (vec) { PICK(4) }
+  PICK(1)
+#undef PICK
+#undef GO
 }

@@ -147,6 +147,8 @@ class Model:
                 self.entries[call.enter[0]].enter(ctx, x, call.enter[1])
             layer.block.forward(ctx, x, layer, cache.binding(i), self.position)
         if ctx.n_want > 0:
+            for part in self.entries:
+                part.close(ctx, x, ctx.want_rows)
             hf = ctx.alloc((ctx.n_want, E), self.rt.act_dtype)
             self.final_norm.forward(ctx, x, hf, rows=ctx.want_rows)
             self.head.forward(ctx, hf, logits_out[:ctx.n_want])

@@ -13,7 +13,7 @@ lower, v, norm, o; latent attention: q, dkv, dkv.norm, uk, uv, o) and `l<i>.mlp.
 """
 from ..config.buborax import BuboraxConfig
 from ..config.registry import register_architecture
-from ..parts.plan import LayerCall, LayerPlan, ModelPlan, PartSpec
+from ..parts.plan import LayerPlan, ModelPlan, PartSpec, looped_order
 
 SLOPE_SPAN = 8.0        # head a's distance penalty is 2^(-SLOPE_SPAN (a + 1) / heads) per position
 
@@ -57,17 +57,11 @@ def build_plan(cfg: BuboraxConfig) -> ModelPlan:
                                 norm2=norm(p + "norm2") if ffn is not None else None, ffn=ffn))
     # the running order: the repeated run of layers `times` times in a row, every call with a cache of
     # its own; the first call of each pass is preceded by the input re-entry with the pass's number
-    entries, order = [], []
-    n, lp = len(cfg.layers), cfg.loop
-    if lp is None:
-        order = [LayerCall(i) for i in range(n)]
-    else:
-        entries.append(PartSpec("input_reentry", {"size": E, "times": lp.times},
+    entries = []
+    if cfg.loop is not None:
+        entries.append(PartSpec("input_reentry", {"size": E, "times": cfg.loop.times},
                                 {"in_weight": "loop.in", "steps": "loop.step"}))
-        order = [LayerCall(i) for i in range(lp.start)]
-        for t in range(lp.times):
-            order += [LayerCall(i, enter=(0, t) if i == lp.start else None) for i in range(lp.start, lp.stop)]
-        order += [LayerCall(i) for i in range(lp.stop, n)]
+    order = looped_order(len(cfg.layers), cfg.loop, enter=0)
     return ModelPlan(
         hidden_size=E, vocab_size=cfg.vocab, max_positions=cfg.max_positions,
         embedding=PartSpec("token_table", {"vocab_size": cfg.vocab, "size": E}, {"table": "embed"}),

@@ -388,7 +388,7 @@ class RotaryAttention(Part):
     heads share; "row_gain": all query heads of a token divided by one root mean square over their
     n_heads x head_dim entries times a gain of that size (`q_norm`), the key heads likewise
     (`k_norm`).  The rotary params may ask for the pairing "neighbours".  `bias`: the four
-    projections have biases.  `own_kv` false: the layer has no key and value projections (nor
+    projections have biases (`out_bias` false: the output projection has none).  `own_kv` false: the layer has no key and value projections (nor
     `k_norm`) and reads what another call cached (the plan's `cache_of`).  `out_mult`: a multiplier
     of the mixer's result (the values are cached times it: the attention is linear in them).
     `sink` "one": a constant 1 in the softmax's denominator (a sink whose score is 0) instead of a
@@ -401,7 +401,7 @@ class RotaryAttention(Part):
     another's keys (for its queries).  `cache_chunk`: the chunk by which the cache may give pages back,
     where a call with another chunk reads them too (default: `chunk`).
     params: size, n_heads, n_kv_heads, head_dim, v_dim, scale, rotary (dims, base, scaling, pairing) or
-    None, qk_norm, eps, chunk, window, sink (false, true or "one"), bias (default false), own_kv (default
+    None, qk_norm, eps, chunk, window, sink (false, true or "one"), bias (default false), out_bias (default: as bias), own_kv (default
     true), out_mult (default 1), gate (None or "entry"), temp (default false), conv (default None),
     cache_chunk."""
 
@@ -413,7 +413,9 @@ class RotaryAttention(Part):
         if own:
             d.update({"k_weight": WeightDecl((G * D, E), "matrix"), "v_weight": WeightDecl((G * V, E), "matrix")})
         if bias:
-            d.update({"q_bias": WeightDecl((H * D,), "bias"), "out_bias": WeightDecl((E,), "bias")})
+            d["q_bias"] = WeightDecl((H * D,), "bias")
+            if params.get("out_bias", True):
+                d["out_bias"] = WeightDecl((E,), "bias")
             if own:
                 d.update({"k_bias": WeightDecl((G * D,), "bias"), "v_bias": WeightDecl((G * V,), "bias")})
         if norm in ("head_gain", "row_gain"):
@@ -458,7 +460,7 @@ class RotaryAttention(Part):
         self.qkv = Linear(store.computed("+".join(r.name for r in refs) + f"+{pad}", lambda: torch.cat(
             [r.tensor.float() for r in refs] + [torch.zeros(pad, refs[0].tensor.shape[1])], 0)), bias)
         out_bias = None
-        if p.get("bias", False):
+        if "out_bias" in tensors:
             ob, m = tensors["out_bias"], self.mult
             out_bias = store.vector(ob) if m == 1.0 else store.computed(
                 f"{ob.name}*{m!r}", kind="vector", make=lambda: (ob.tensor.double() * m).float())

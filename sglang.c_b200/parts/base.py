@@ -22,6 +22,10 @@ Interfaces by category (ctx is an `engine.step.StepContext`):
                                                  residual += ff(h), or out = ff(h)
   stream_mix    begin(ctx, x) / finish(ctx, x)   around a layer: x becomes a mix of this and
                                                  earlier layers' results (kept in ctx.shared)
+                start(ctx, x) / close(ctx, x, rows)
+                                                 (a plan's `entries`) after the embedding; after the
+                                                 last layer, where x[rows] must hold what the final
+                                                 norm reads
   token_mix     forward(ctx, x, norm1, h1, norm2, h2, cache)
                                                  h1 = norm1(x) mixed with earlier tokens' (kept in
                                                  `cache`), h2 = norm2(x) (or norm2, h2 None)
@@ -66,6 +70,9 @@ class Part:
         block gets its built layer as argument and answers for the whole layer).  The engine
         sizes the step workspace from the answers."""
         return 0
+
+    def close(self, ctx, x, rows):
+        """Parts of a plan's `entries`: leave in x[rows] (rows int32) what the final norm reads."""
 
     def graph_bound(self, ctx):
         """Mixers only: an upper bound of the context length for this step's launches, if the

@@ -35,6 +35,38 @@ class PreNormBlock(Part):
         return x
 
 
+@register_part("block", "stream_pre_norm")
+class StreamPreNormBlock(Part):
+    """The pre-norm arrangement over several residual streams: each sublayer reads the norm of one
+    combination of the streams and writes its result back into all of them, as the layer's sub-parts
+    `hc1` (mixer) and `hc2` (feed-forward) of category stream_mix say.  The streams themselves belong to
+    the model's `residual_streams` part; the write of a sublayer is done by the launch that makes the next
+    one's input.  The second sublayer is there only if the layer has an `ffn`."""
+
+    def workspace_per_token(self, layer):
+        inner = layer.mixer.workspace_per_token()
+        if "ffn" in layer.parts:
+            inner = max(inner, layer.ffn.workspace_per_token())
+        return inner
+
+    def forward(self, ctx, x, layer, cache, position=None):
+        streams = ctx.shared["residual_streams"]
+        for norm in (layer.norm1, layer.parts.get("norm2")):
+            if norm is not None and (norm.form != "rms" or norm.bias is not None or norm.groups != 1):
+                raise ValueError("stream_pre_norm: the norms are plain RMS norms")
+        mark = ctx.mark()
+        h = streams.read(ctx, layer.hc1, layer.norm1)
+        layer.mixer.forward(ctx, h, residual=None, cache=cache, position=position, out=streams.y)
+        streams.written(layer.hc1)
+        ctx.release(mark)
+        if "ffn" in layer.parts:
+            h = streams.read(ctx, layer.hc2, layer.norm2)
+            layer.ffn.forward(ctx, h, residual=None, out=streams.y)
+            streams.written(layer.hc2)
+            ctx.release(mark)
+        return x
+
+
 @register_part("block", "sandwich_norm")
 class SandwichNormBlock(Part):
     """A norm ahead of and a norm behind each sublayer:

@@ -75,8 +75,10 @@ class GatedMLP(Part):
     product; the gating runs on its result; the down projection adds into the stream.  The
     multiplier m of the sublayer's result is taken by the gating kernel, in 32-bit, ahead of the
     down projection (which is linear), so a model with m != 1 and a down bias is not served.
-    params: size, inner_size, bias, activation ("silu", the default, or "gelu_tanh"), out_mult (m,
-    default 1)."""
+    With activation "clamped" gate and up values are bounded first and the gate's function has a slope:
+    g = min(gate, limit), u = clamp(up, -limit, limit), and g sigmoid(slope g) (u + 1) takes the place of act(.) u.
+    params: size, inner_size, bias, activation ("silu", the default, "gelu_tanh" or "clamped"), slope and
+    limit ("clamped" only), out_mult (m, default 1)."""
 
     def __init__(self, params, runtime):
         super().__init__(params, runtime)
@@ -117,7 +119,8 @@ class GatedMLP(Part):
         gu = ctx.alloc((T, 2 * F), self.rt.act_dtype)
         self.gate_up.forward(ctx, h, out=gu)
         z = ctx.alloc((T, F), self.rt.act_dtype)
-        ops.gated_act(gu, z, act=self.params.get("activation", "silu"), mult=float(self.params.get("out_mult", 1.0)))
+        ops.gated_act(gu, z, act=self.params.get("activation", "silu"), mult=float(self.params.get("out_mult", 1.0)),
+                      slope=self.params.get("slope"), limit=self.params.get("limit"))
         return self.down.forward(ctx, z, out=out, residual=residual)
 
 

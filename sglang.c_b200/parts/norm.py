@@ -24,7 +24,13 @@ class LayerNorm(Part):
 
     def load(self, tensors, store):
         ref = tensors["weight"]
-        if self.params.get("one_plus"):
+        m = float(self.params.get("out_mult", 1.0))
+        if m != 1.0:
+            if "bias" in tensors or self.params.get("one_plus"):
+                raise ValueError("a norm's result multiplier goes with a plain gain and no bias")
+            self.weight = store.computed(f"{ref.name}*{m!r}", kind="vector",
+                                         make=lambda: (ref.tensor.double() * m).float())
+        elif self.params.get("one_plus"):
             # a gain stored around zero: the kernels multiply by 1 + w, formed once
             self.weight = store.computed(ref.name + "+1", kind="vector", make=lambda: ref.tensor.float() + 1.0)
         else:
@@ -86,7 +92,8 @@ class RMSNorm(LayerNorm):
     """y = x / sqrt(mean(x^2) + eps) * weight, eps inside the root, statistics in 32-bit.
     params: size, eps, groups (default 1; more: each of so many equal consecutive parts of the row is
     divided by its own root mean square), one_plus (default false; true: the file's tensor is stored
-    around zero and the gain is 1 + it)."""
+    around zero and the gain is 1 + it), out_mult (default 1: a multiplier of the result, folded into the
+    gain)."""
 
     form = "rms"
 

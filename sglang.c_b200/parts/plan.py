@@ -92,6 +92,19 @@ class LayerCall:
     enter: Optional[Tuple[int, int]] = None
 
 
+def looped_order(n_layers, loop, enter=None):
+    """The running order of n_layers layers of which a run repeats: `loop` (start, stop, times as
+    attributes, or None) has layers start .. stop-1 run `times` times in a row, every call with a cache of its
+    own; `enter`: the entry part (an index) ahead of each pass."""
+    if loop is None:
+        return [LayerCall(i) for i in range(n_layers)]
+    order = [LayerCall(i) for i in range(loop.start)]
+    for t in range(loop.times):
+        order += [LayerCall(i, enter=(enter, t) if i == loop.start and enter is not None else None)
+                  for i in range(loop.start, loop.stop)]
+    return order + [LayerCall(i) for i in range(loop.stop, n_layers)]
+
+
 @dataclass
 class ModelPlan:
     hidden_size: int
@@ -109,7 +122,8 @@ class ModelPlan:
     # prefixes to try when a name is not found as written
     name_prefixes: Tuple[str, ...] = ("",)
     # parts of category stream_mix that act between layers: each sees the embedding output
-    # (`start(ctx, x)`) and runs where a LayerCall's `enter` names it
+    # (`start(ctx, x)`), runs where a LayerCall's `enter` names it, and is asked once more behind the
+    # last layer (`close(ctx, x, rows)`)
     entries: List[PartSpec] = field(default_factory=list)
 
     def part_specs(self):

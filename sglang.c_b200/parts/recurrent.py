@@ -406,3 +406,74 @@ class MatrixMemory(Part):
         ops.gated_norm(o, ctx.columns(pre, c_g, c_i), self.norm, y, H, V, float(p["eps"]), "sigmoid", o_pitch=V + 1,
                        m_run=m_run)
         return self.out.forward(ctx, y, out=out, residual=residual)
+
+
+@register_part("mixer", "mamba2")
+class SelectiveStateSpace(Part):
+    """A selective state space with one decay per head and token (Mamba-2).  One projection of h is laid out
+    [z | x | B | C | dt] (n_heads v_dim, n_heads v_dim, n_groups dim, n_groups dim, n_heads columns);
+    x, B and C pass a causal convolution of `conv` taps over time per channel, with a bias, and silu;
+    dt = softplus(dt + dt_bias); per head (head i reads B and C of group i / (n_heads / n_groups))
+        S <- exp(-exp(A_log) dt) S + dt B x^T,   y = S^T C + D x         (S [dim x v_dim]);
+    the heads' y side by side times silu(z), RMS-normed in norm_groups equal parts (eps) with a gain of
+    n_heads v_dim entries, then projected.  The projection leaves its product in 32-bit; convolution, dt
+    and decays, state, gate and norm are 32-bit.  Kept per request: S, and the last conv - 1 inputs
+    of the convolution.
+    params: size, n_heads, v_dim, dim, n_groups, conv, norm_groups, eps."""
+
+    @classmethod
+    def declare_weights(cls, params):
+        E, H, V, N, G, K = (params[k] for k in ("size", "n_heads", "v_dim", "dim", "n_groups", "conv"))
+        C = H * V + 2 * G * N
+        return {"in_weight": WeightDecl((H * V + C + H, E), "matrix"), "conv": WeightDecl((C, K), "conv_taps"),
+                "conv_bias": WeightDecl((C,), "bias"), "dt_bias": WeightDecl((H,), "bias"),
+                "A_log": WeightDecl((H,), "bias"), "D": WeightDecl((H,), "norm_gain"),
+                "norm": WeightDecl((H * V,), "norm_gain"), "out_weight": WeightDecl((E, H * V), "residual_matrix")}
+
+    def load(self, tensors, store):
+        p = self.params
+        if p["n_heads"] % p["n_groups"] or (p["n_heads"] * p["v_dim"]) % p["norm_groups"]:
+            raise ValueError("mamba2: heads split into n_groups, their results into norm_groups equal parts")
+        w = tensors["in_weight"]
+        pad = (-w.tensor.shape[0]) % 8
+        self.inp = Linear(store.computed(f"{w.name}+{pad}", lambda: torch.cat(
+            [w.tensor.float(), torch.zeros(pad, w.tensor.shape[1])], 0)), None)
+        taps = tensors["conv"]             # [taps, channels]: a tap's channels lie side by side
+        self.taps = store.computed(taps.name + ".T", kind="vector", make=lambda: taps.tensor.float().t())
+        self.conv_bias, self.dt_bias, self.A_log, self.D, self.norm = (
+            store.vector(tensors[k]) for k in ("conv_bias", "dt_bias", "A_log", "D", "norm"))
+        self.out = Linear(store.matrix(tensors["out_weight"]), None)
+
+    def _channels(self):
+        p = self.params
+        return p["n_heads"] * p["v_dim"] + 2 * p["n_groups"] * p["dim"]
+
+    def cache_need(self):
+        p = self.params
+        return (CacheNeed.state((p["n_heads"], p["dim"], p["v_dim"]), "float32"),
+                CacheNeed.state((max(p["conv"] - 1, 0), self._channels()), "float32"))
+
+    def workspace_per_token(self):
+        p = self.params
+        inner, C = p["n_heads"] * p["v_dim"], self._channels()
+        act = 4 if self.rt.dtype == "float32" else 2
+        return 4 * (2 * inner + 2 * C + 3 * p["n_heads"] + 8) + act * inner + 2048
+
+    def forward(self, ctx, h, residual, cache, position=None, out=None):
+        p = self.params
+        H, V, N, G = p["n_heads"], p["v_dim"], p["dim"], p["n_groups"]
+        T, inner, C, parts = h.shape[0], H * V, self._channels(), p["norm_groups"]
+        state, tail = cache
+        pre = ctx.alloc((T, self.inp.out_size), torch.float32)
+        self.inp.forward(ctx, h, out=pre)
+        u = ctx.alloc((T, C), torch.float32)
+        gates = ctx.alloc((T, 2 * H), torch.float32)
+        ops.conv_silu(ctx.columns(pre, inner, inner + C + H), self.taps, self.conv_bias, tail.tensor, u, ctx.token_req,
+                      ctx.q_start, ctx.state_slots, ctx.R, gates=(H, C, self.A_log, self.dt_bias, gates))
+        y = ctx.alloc((T, inner), torch.float32)
+        ops.matrix_state("gated", ctx.columns(u, inner + G * N, C), ctx.columns(u, inner, inner + G * N),
+                         ctx.columns(u, 0, inner), y, state.tensor, ctx.q_start, ctx.state_slots, ctx.R, H, G, N, V,
+                         gates=gates, skip=self.D)
+        z = ctx.alloc((T, inner), self.rt.act_dtype)
+        ops.gate_then_norm(y, ctx.columns(pre, 0, inner), self.norm, z, parts, inner // parts, float(p["eps"]), "silu")
+        return self.out.forward(ctx, z, out=out, residual=residual)

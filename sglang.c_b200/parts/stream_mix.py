@@ -130,3 +130,65 @@ class TokenGatedInput(Part):
             if cast_out is not None:
                 ops.cast_rows(x[:T], cast_out)
         return x
+
+
+@register_part("stream_mix", "residual_streams")
+class ResidualStreams(Part):
+    """Several residual streams side by side (hyper-connections): copies of the embedding output at the
+    start, their sum at the end.  `start` takes the streams' buffer [T, streams, size], one for a
+    sublayer's result and one for what a sublayer reads from the step workspace, below the layers'
+    buffers; the block `stream_pre_norm` works on them through `read` and `written`.  What a sublayer made goes
+    into the streams in the launch that makes the next sublayer's input (ops.stream_step), so `close`,
+    behind the last layer, does the last write and the sum, for the rows whose logits are asked for.
+    params: size, streams."""
+
+    KEY = "residual_streams"
+
+    def load(self, tensors, store):
+        n = self.params["streams"]
+        self.ones = store.computed(f"ones:{n}", kind="vector", make=lambda: torch.ones(n))
+
+    def workspace_per_token(self):
+        act = 4 if self.rt.dtype == "float32" else 2
+        return (4 * (self.params["streams"] + 1) + act) * self.params["size"] + 1024
+
+    def start(self, ctx, x):
+        T, E, S = x.shape[0], self.params["size"], self.params["streams"]
+        self.streams = ctx.alloc((T, S, E), torch.float32)
+        self.y = ctx.alloc((T, E), torch.float32)
+        self.h = ctx.alloc((T, E), self.rt.act_dtype)
+        self.source = x.unsqueeze(1).expand(T, S, E)       # before the first write: copies of one row
+        self.pending = None
+        ctx.shared[self.KEY] = self
+
+    def read(self, ctx, hc, norm):
+        """The rows the next sublayer works on: norm(sum_s in[s] X_s), after the write that is still due."""
+        write = None
+        if self.pending is not None:
+            write = (self.y, self.pending.w_out, self.pending.w_mix, self.streams)
+        ops.stream_step(self.source, self.h, hc.w_in, norm.weight, float(norm.params["eps"]), write=write)
+        if write is not None:
+            self.source, self.pending = self.streams, None
+        return self.h
+
+    def written(self, hc):
+        """The sublayer's result is in self.y; it goes into the streams as `hc` says."""
+        self.pending = hc
+
+    def close(self, ctx, x, rows):
+        write = (self.y, self.pending.w_out, self.pending.w_mix, None) if self.pending is not None else None
+        ops.stream_step(self.source, x, self.ones, write=write, rows=rows)
+
+
+@register_part("stream_mix", "stream_connection")
+class StreamConnection(Part):
+    """How one sublayer is tied to the residual streams: it reads sum_s in[s] X_s, and its result y goes back
+    as X_t <- sum_s mix[s, t] X_s + out[t] y (mix is indexed [from, to]).  params: streams."""
+
+    @classmethod
+    def declare_weights(cls, params):
+        n = params["streams"]
+        return {"in": WeightDecl((n,), "norm_gain"), "out": WeightDecl((n,), "norm_gain"), "mix": WeightDecl((n, n), "mixing")}
+
+    def load(self, tensors, store):
+        self.w_in, self.w_out, self.w_mix = (store.vector(tensors[k]) for k in ("in", "out", "mix"))
