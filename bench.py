@@ -18,7 +18,7 @@ requests) over its time, against the measured copy bandwidth; `points` has decod
 at batch 1 and 64, the true 32-bit path and the prefill through the C interface;
 `kernels` says where a decode and a
 prefill step's time goes, kernel by kernel.  `--full` adds medium and XL layer
-sizes and the mixed workload to `points`.  `--compare tukavik` (or `zuretar`, or `buborax`, each of which adds its design as one more column; `lubavik`: that design beside Zuretar, the closest one; `fupapel`: that design beside Lubavik, the closest, and Tukavik for its latents) measures,
+sizes and the mixed workload to `points`.  `--compare tukavik` (or `zuretar`, or `buborax`, each of which adds its design as one more column; `lubavik`: that design beside Zuretar, the closest one; `fupapel`: that design beside Lubavik, the closest, and Tukavik for its latents; `zadunex`: that design beside Zuretar and Lubavik, the closest) measures,
 instead of all this, a Tukavik model beside the GPT-2 model of the same layer sizes.
 """
 import argparse
@@ -966,6 +966,62 @@ def fupapel_step_bytes(cfg, batch, context, prompt_tokens):
     return out
 
 
+def zadunex_config(base, n_layer):
+    """A Zadunex model with the layer sizes of a GPT-2 model: the same width, number of layer runs, head
+    size (64) and vocabulary, four residual streams.  Layers in fours: a state space of twice the width (twice
+    the model's heads of 64 over a state of 128 rows, one group, four taps) with a gated feed-forward of two
+    thirds the width of GPT-2's; attention (the model's heads over a quarter as many key/value heads, half of
+    each head turned) with a mixture of 8 experts of a sixth of that width, 2 chosen; and the state space
+    twice more, with the experts each.  Layers 1 and 2 run twice, so the file holds two layers fewer than run."""
+    E, H, I = base["n_embd"], base["n_head"], base["n_inner"]
+    dense = {"kind": "dense", "ff": max(64, (2 * I // 3) // 64 * 64), "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": max(64, (I // 6) // 64 * 64)}, "router": {"experts": 8, "top": 2}}
+    space = {"heads": 2 * H, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    attn = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 64, "scale": 0.125, "rot": {"base": 10000.0, "dims": 32}}
+    kinds = [("mamba2", space, dense), ("attention", attn, moe), ("mamba2", space, moe), ("mamba2", space, moe)]
+    layers = [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(max(3, n_layer - 2))]
+    return {"architecture": "Zadunex", "vocab": base["vocab_size"], "width": E, "streams": 4, "norm": {"eps": 1e-6},
+            "logit_scale": 1.0, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers,
+            "max_positions": base["n_positions"]}
+
+
+def zadunex_step_bytes(cfg, batch, context, prompt_tokens):
+    """What the kernels that this design adds or extends must move in a step (32-bit streams, projections
+    and states; bfloat16 activations and cache): {decode | prefill: {kernel label: bytes}}.  The recurrence
+    in chunks is counted like the one token by token: its inputs, its results and the requests' states once."""
+    lp = cfg["loop"]
+    runs = list(range(lp["start"])) + list(range(lp["start"], lp["stop"])) * lp["times"] + \
+        list(range(lp["stop"], len(cfg["layers"])))
+    E, S = cfg["width"], cfg["streams"]
+    out = {}
+    for name, T, R in (("decode", batch, batch), ("prefill", prompt_tokens, 2)):
+        step = conv = state = gnorm = prep = attn = gact = route = 0
+        for i in runs:
+            layer = cfg["layers"][i]
+            m, mlp = layer["mixer"], layer["mlp"]
+            step += 2 * T * E * ((2 * S + 1) * 4 + 2)          # the streams read and written, the result, the next rows
+            if layer["type"] == "mamba2":
+                H, V, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+                inner, C = H * V, H * V + 2 * G * N
+                conv += T * (2 * C + 3 * H) * 4 + R * (m["conv"] - 1) * C * 8
+                state += R * H * N * V * 8 + T * (C + inner + H) * 4
+                gnorm += T * inner * (8 + 2)
+            else:
+                H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+                prep += T * (H * D + G * (D + V)) * (4 + 2)
+                if name == "decode":
+                    attn += T * context * G * (D + V) * 2 + T * H * (D + V) * 2
+            if mlp["kind"] == "dense":
+                gact += T * mlp["ff"] * 6
+            else:
+                X = mlp["router"]["experts"]
+                gact += T * mlp["expert"]["ff"] * X * 6 + T * X * 4
+                route += T * X * 8 + T * mlp["router"]["top"] * 8
+        out[name] = {"stream_step": step, "conv_silu": conv, "matrix_state": state, "gate_then_norm": gnorm, "qk_prep": prep,
+                     "attention_ext": attn, "gated_act": gact, "router": route}
+    return out
+
+
 DESIGNS = {"tukavik": (tukavik_config, tukavik_step_bytes,
                        {"mingru_scan": "mingru_scan", "norm_rows": "norm_rows", "depth_mix": "depth_mix",
                         "attention_decode_shared": "attention_shared"}),
@@ -979,7 +1035,10 @@ DESIGNS = {"tukavik": (tukavik_config, tukavik_step_bytes,
                                        "gated_act", "norm_add_tail", "gated_gather", "router")}),
            "fupapel": (fupapel_config, fupapel_step_bytes,
                        {k: k for k in ("norm_pair_shift", "qk_prep", "short_conv_tail", "latent_rope", "attention_ext",
-                                       "attention_latent_decode", "gated_act", "router")})}
+                                       "attention_latent_decode", "gated_act", "router")}),
+           "zadunex": (zadunex_config, zadunex_step_bytes,
+                       dict({k: k for k in ("stream_step", "conv_silu", "matrix_state", "gate_then_norm", "qk_prep",
+                                            "attention_ext", "gated_act", "router")}, state_chunks="matrix_state"))}
 
 
 def compare_designs(designs, sizes, steps, warmup, pk):
@@ -1108,7 +1167,7 @@ def main():
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "fp32"],
                     help="a handful of steps of one kind and nothing else (what a profiler is pointed at): "
                          "decode steps at batch 8, prefill steps of 2 x 1,024 tokens, or both on the 32-bit path")
-    ap.add_argument("--compare", default=None, choices=["tukavik", "zuretar", "buborax", "lubavik", "fupapel"],
+    ap.add_argument("--compare", default=None, choices=["tukavik", "zuretar", "buborax", "lubavik", "fupapel", "zadunex"],
                     help="nothing of the above: decode and prefill of a model of this design beside the GPT-2 model "
                          "of equal layer sizes (--model, or small and medium with --full), with both kernel tables")
     args = ap.parse_args()
@@ -1130,7 +1189,7 @@ def main():
         clocks.start()
         designs = {"tukavik": ["tukavik"], "zuretar": ["tukavik", "zuretar"],
                    "buborax": ["tukavik", "zuretar", "buborax"], "lubavik": ["zuretar", "lubavik"],
-                   "fupapel": ["tukavik", "lubavik", "fupapel"]}[args.compare]
+                   "fupapel": ["tukavik", "lubavik", "fupapel"], "zadunex": ["zuretar", "lubavik", "zadunex"]}[args.compare]
         res = compare_designs(designs, ["small", "medium"] if args.full else [args.model], steps, warmup, pk)
         print(json.dumps({"metric": f"decode and prefill tok/s, {' and '.join(d.capitalize() for d in designs)} beside "
                                     "GPT-2 at equal layer sizes (Python engine)",

@@ -1068,6 +1068,60 @@ def matrix_state(mode, q, k, v, out, state, q_start, state_slots, n_requests, n_
     _check(lib, code, f"matrix_state ({mode}, {dim} x {v_dim})")
 
 
+STATE_CHUNK = 64            # tokens of a chunk (state_chunks.cu: SC_Q)
+STATE_CHUNK_MIN_LEN = 64    # a step whose longest portion has fewer tokens goes token by token
+
+
+def state_chunks_pay(n_tokens, n_requests, max_q_len):
+    """Whether a step's recurrence is worked on in chunks: long portions, and not many short ones beside
+    them (a chunk has a fixed cost, and the workspace holds a state per chunk)."""
+    return max_q_len >= STATE_CHUNK_MIN_LEN and n_requests <= n_tokens // STATE_CHUNK
+
+
+def state_chunks_workspace(n_tokens, n_requests, n_heads, n_groups, dim, v_dim):
+    """Floats of workspace that state_chunks takes for such a step (at most twice the whole chunks that
+    fit into n_tokens where state_chunks_pay holds)."""
+    return (n_tokens // STATE_CHUNK + n_requests) * (n_heads * dim * v_dim + n_groups * STATE_CHUNK ** 2 + n_heads)
+
+
+def state_chunks(q, k, v, weights, A_log, out, state, q_start, state_slots, n_requests, n_heads, n_groups, dim, v_dim,
+                 workspace, skip=None):
+    """matrix_state's gated form in chunks that run side by side (state_chunks.cu), for portions of
+    many tokens, where the decay is made from the input weight: S <- exp(-exp(A_log_h) b) S + b k v^T,
+    o = S^T q + skip_h v.  weights: float32 [T, >= H], the first H columns are b; A_log, skip (or None):
+    float32 [H]; the rest as matrix_state's; workspace: float32, state_chunks_workspace entries."""
+    _need_cuda(q, k, v, weights, A_log, out, state, q_start, state_slots, workspace, skip)
+    T = out.shape[0]
+    _f32_rows(q, "state_chunks: q", n_groups * dim)
+    _f32_rows(k, "state_chunks: k", n_groups * dim)
+    _f32_rows(v, "state_chunks: v", n_heads * v_dim)
+    _f32_rows(out, "state_chunks: out", n_heads * v_dim)
+    _f32_rows(weights, "state_chunks: weights")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (n_heads, dim, v_dim):
+        raise KernelError(f"state_chunks: the state is float32 [n_slots, {n_heads}, {dim}, {v_dim}]")
+    if weights.shape[1] < n_heads or min(t.shape[0] for t in (q, k, v, weights)) < T:
+        raise KernelError("state_chunks: a row of q, k, v and weights for every token")
+    for t, nm in ((A_log, "A_log"), (skip, "skip")):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != n_heads or not t.is_contiguous()):
+            raise KernelError(f"state_chunks: {nm} is a float32 number per head")
+    _i32(q_start, "q_start")
+    _i32(state_slots, "state_slots")
+    n_chunks = T // STATE_CHUNK + int(n_requests)
+    if workspace.dtype != torch.float32 or not workspace.is_contiguous() \
+            or workspace.numel() < state_chunks_workspace(T, int(n_requests), n_heads, n_groups, dim, v_dim):
+        raise KernelError("state_chunks: the workspace is too small")
+    lib = build.load("state_chunks")
+    if lib.sglc_state_chunk() != STATE_CHUNK:
+        raise KernelError("state_chunks: the library's chunk size differs from the binding's")
+    code = lib.sglc_state_chunks(_ptr(q), ctypes.c_longlong(q.stride(0)), _ptr(k), ctypes.c_longlong(k.stride(0)), _ptr(v),
+                                 ctypes.c_longlong(v.stride(0)), _ptr(weights), ctypes.c_longlong(weights.stride(0)),
+                                 _ptr(A_log), _ptr(skip), _ptr(out), ctypes.c_longlong(out.stride(0)), _ptr(state),
+                                 state.shape[0], _ptr(q_start), _ptr(state_slots), int(n_requests), int(n_heads),
+                                 int(n_groups), int(dim), int(v_dim), _ptr(workspace), n_chunks,
+                                 _ptr(tc_error_flag(q.device)), _stream())
+    _check(lib, code, f"state_chunks ({dim} x {v_dim})", n_kernels=3)
+
+
 def gated_norm(o, gate, gain, y, groups, width, eps, act, o_pitch=None, m_run=None):
     """y = o / sqrt(mean(o^2) + eps) * gain * act(gate) per row of `width` (a token has `groups`
     rows side by side; gain float32 [width] serves them all, or [groups*width] every row its own);

@@ -457,7 +457,8 @@ class SelectiveStateSpace(Part):
         p = self.params
         inner, C = p["n_heads"] * p["v_dim"], self._channels()
         act = 4 if self.rt.dtype == "float32" else 2
-        return 4 * (2 * inner + 2 * C + 3 * p["n_heads"] + 8) + act * inner + 2048
+        chunks = ops.state_chunks_workspace(ops.STATE_CHUNK, 1, p["n_heads"], p["n_groups"], p["dim"], p["v_dim"])
+        return 4 * (2 * inner + 2 * C + 3 * p["n_heads"] + 8) + act * inner + 2048 + 4 * chunks // ops.STATE_CHUNK
 
     def forward(self, ctx, h, residual, cache, position=None, out=None):
         p = self.params
@@ -471,9 +472,17 @@ class SelectiveStateSpace(Part):
         ops.conv_silu(ctx.columns(pre, inner, inner + C + H), self.taps, self.conv_bias, tail.tensor, u, ctx.token_req,
                       ctx.q_start, ctx.state_slots, ctx.R, gates=(H, C, self.A_log, self.dt_bias, gates))
         y = ctx.alloc((T, inner), torch.float32)
-        ops.matrix_state("gated", ctx.columns(u, inner + G * N, C), ctx.columns(u, inner, inner + G * N),
-                         ctx.columns(u, 0, inner), y, state.tensor, ctx.q_start, ctx.state_slots, ctx.R, H, G, N, V,
-                         gates=gates, skip=self.D)
+        qkv = ctx.columns(u, inner + G * N, C), ctx.columns(u, inner, inner + G * N), ctx.columns(u, 0, inner)
+        # long portions in chunks side by side, everything else token by token
+        if ops.state_chunks_pay(T, ctx.R, ctx.max_q_len):
+            inner_mark = ctx.mark()
+            ws = ctx.alloc((ops.state_chunks_workspace(T, ctx.R, H, G, N, V),), torch.float32)
+            ops.state_chunks(*qkv, gates, self.A_log, y, state.tensor, ctx.q_start, ctx.state_slots, ctx.R, H, G, N, V, ws,
+                             skip=self.D)
+            ctx.release(inner_mark)
+        else:
+            ops.matrix_state("gated", *qkv, y, state.tensor, ctx.q_start, ctx.state_slots, ctx.R, H, G, N, V, gates=gates,
+                             skip=self.D)
         z = ctx.alloc((T, inner), self.rt.act_dtype)
         ops.gate_then_norm(y, ctx.columns(pre, 0, inner), self.norm, z, parts, inner // parts, float(p["eps"]), "silu")
         return self.out.forward(ctx, z, out=out, residual=residual)
