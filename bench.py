@@ -1038,7 +1038,7 @@ DESIGNS = {"tukavik": (tukavik_config, tukavik_step_bytes,
                                        "attention_latent_decode", "gated_act", "router")}),
            "zadunex": (zadunex_config, zadunex_step_bytes,
                        dict({k: k for k in ("stream_step", "conv_silu", "matrix_state", "gate_then_norm", "qk_prep",
-                                            "attention_ext", "gated_act", "router")}, state_chunks="matrix_state"))}
+                                            "attention_ext", "gated_act", "router")}, state_chunks="matrix_state", state_step="matrix_state"))}
 
 
 def compare_designs(designs, sizes, steps, warmup, pk):

@@ -1122,6 +1122,32 @@ def state_chunks(q, k, v, weights, A_log, out, state, q_start, state_slots, n_re
     _check(lib, code, f"state_chunks ({dim} x {v_dim})", n_kernels=3)
 
 
+def state_step(q, k, v, gates, out, state, state_slots, n_heads, n_groups, dim, v_dim, skip=None):
+    """matrix_state's gated form (with its skip) for a step in which every request brings one token: row r
+    is request r's.  gates: float32 [R, 2H] (input weights, decays)."""
+    _need_cuda(q, k, v, gates, out, state, state_slots, skip)
+    R = out.shape[0]
+    _f32_rows(q, "state_step: q", n_groups * dim)
+    _f32_rows(k, "state_step: k", n_groups * dim)
+    _f32_rows(v, "state_step: v", n_heads * v_dim)
+    _f32_rows(out, "state_step: out", n_heads * v_dim)
+    _f32_rows(gates, "state_step: gates", 2 * n_heads)
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (n_heads, dim, v_dim):
+        raise KernelError(f"state_step: the state is float32 [n_slots, {n_heads}, {dim}, {v_dim}]")
+    if skip is not None and (skip.dtype != torch.float32 or skip.numel() != n_heads or not skip.is_contiguous()):
+        raise KernelError("state_step: skip is a float32 factor per head")
+    _i32(state_slots, "state_slots")
+    if state_slots.numel() < R or min(t.shape[0] for t in (q, k, v, gates)) < R:
+        raise KernelError("state_step: a slot and a row of q, k, v and gates for every request")
+    lib = build.load("state_chunks")
+    code = lib.sglc_state_step(_ptr(q), ctypes.c_longlong(q.stride(0)), _ptr(k), ctypes.c_longlong(k.stride(0)), _ptr(v),
+                               ctypes.c_longlong(v.stride(0)), _ptr(gates), _ptr(gates[:, n_heads:]),
+                               ctypes.c_longlong(gates.stride(0)), _ptr(skip), _ptr(out), ctypes.c_longlong(out.stride(0)),
+                               _ptr(state), state.shape[0], _ptr(state_slots), R, int(n_heads), int(n_groups), int(dim),
+                               int(v_dim), _ptr(tc_error_flag(q.device)), _stream())
+    _check(lib, code, f"state_step ({dim} x {v_dim})")
+
+
 def gated_norm(o, gate, gain, y, groups, width, eps, act, o_pitch=None, m_run=None):
     """y = o / sqrt(mean(o^2) + eps) * gain * act(gate) per row of `width` (a token has `groups`
     rows side by side; gain float32 [width] serves them all, or [groups*width] every row its own);

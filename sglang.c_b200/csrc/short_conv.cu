@@ -189,7 +189,7 @@ SGLC_API int sglc_short_conv_tail(const float* x, long long x_stride, float* tai
 }
 
 // y_t[ch] = silu(bias[ch] + sum_j taps[j][ch] x_{t-(K-1)+j}[ch]): a thread takes CW neighbouring channels of
-// `per` consecutive tokens of the step and moves a window over them.  Tails in the same launch: the
+// `per` consecutive tokens of the step.  Tails in the same launch: the
 // tokens that look back before their portion, its first K-1, all belong to the thread that meets the portion's
 // first token (others pass over them), so a channel's tail has one reader, which then moves it on.
 // The last row of blocks makes the gates.
@@ -205,6 +205,8 @@ struct ConvSiluArgs {
   float* gates; long long gates_stride;     // [T][2 heads]: dt, then the decay
   int* err;
 };
+
+constexpr int CONV_PER = 8;
 
 template <int CW> struct ConvVec;
 template <> struct ConvVec<1> {
@@ -225,8 +227,8 @@ template <> struct ConvVec<4> {
   __device__ ConvVec silu() const { return {make_float4(silu_f32(v.x), silu_f32(v.y), silu_f32(v.z), silu_f32(v.w))}; }
 };
 
-// KT: the taps as a constant (the window then stays in registers), or 0: any number, inputs read again.
-template <int CW, int KT>
+// KT: the taps as a constant, or 0: any number.  PER: the tokens of a thread as a constant, or 1.
+template <int CW, int KT, int PER>
 __global__ void __launch_bounds__(128)
 conv_silu_kernel(const ConvSiluArgs p) {
   using V = ConvVec<CW>;
@@ -245,7 +247,7 @@ conv_silu_kernel(const ConvSiluArgs p) {
   const int ch = (blockIdx.y * 128 + threadIdx.x) * CW;
   if (ch >= p.C) return;
   const int K = KT ? KT : p.K;
-  V w[KT ? KT : 1], win[KT > 1 ? KT - 1 : 1];
+  V w[KT ? KT : 1];
   if constexpr (KT > 0) {
 #pragma unroll
     for (int j = 0; j < KT; j++) w[j] = V::load(p.taps + (size_t)j * p.C + ch);
@@ -253,12 +255,26 @@ conv_silu_kernel(const ConvSiluArgs p) {
   const V b = V::load(p.bias + ch);
   const float* x = p.x + ch;
   pdl_wait();
-  bool have = false;                         // the window holds the K-1 inputs ahead of token t
+  int r = p.token_req[ta], q0 = p.q_start[r], q1 = p.q_start[r + 1];
+  if constexpr (KT > 0 && PER > 1) {         // tokens of one request, past its first ones: every input is asked for at once
+    if (tb - ta == PER && q1 >= tb && ta - q0 >= KT - 1) {
+      V in[PER + KT - 1];
+#pragma unroll
+      for (int e = 0; e < PER + KT - 1; e++) in[e] = V::load(x + (size_t)(ta - (KT - 1) + e) * p.x_stride);
+#pragma unroll
+      for (int e = 0; e < PER; e++) {
+        V a = b;
+#pragma unroll
+        for (int j = 0; j < KT; j++) a.fma(w[j], in[e + j]);
+        a.silu().store(p.y + (size_t)(ta + e) * p.y_stride + ch);
+      }
+      return;
+    }
+  }
   for (int t = ta; t < tb; t++) {
-    const int r = p.token_req[t];
-    const int q0 = p.q_start[r], i = t - q0;
+    while (t >= q1) { r++; q0 = q1; q1 = p.q_start[r + 1]; }      // (a request without tokens ends where it begins)
+    const int i = t - q0;
     if (i < K - 1) {
-      have = false;
       if (i > 0) continue;                   // (done with the portion's first token)
       const int n = p.q_start[r + 1] - q0;
       const int slot = p.state_slots[r];
@@ -280,23 +296,8 @@ conv_silu_kernel(const ConvSiluArgs p) {
       continue;
     }
     V a = b;
-    if constexpr (KT > 0) {
-      if (!have) {
-#pragma unroll
-        for (int j = 0; j < KT - 1; j++) win[j] = V::load(x + (size_t)(t - (KT - 1) + j) * p.x_stride);
-        have = true;
-      }
-      const V now = V::load(x + (size_t)t * p.x_stride);
-#pragma unroll
-      for (int j = 0; j < KT - 1; j++) a.fma(w[j], win[j]);
-      a.fma(w[KT - 1], now);
-#pragma unroll
-      for (int j = 0; j + 1 < KT - 1; j++) win[j] = win[j + 1];
-      if constexpr (KT > 1) win[KT - 2] = now;
-    } else {
-      for (int j = 0; j < K; j++)
-        a.fma(V::load(p.taps + (size_t)j * p.C + ch), V::load(x + (size_t)(t - (K - 1) + j) * p.x_stride));
-    }
+    for (int j = 0; j < K; j++)
+      a.fma(V::load(p.taps + (size_t)j * p.C + ch), V::load(x + (size_t)(t - (K - 1) + j) * p.x_stride));
     a.silu().store(p.y + (size_t)t * p.y_stride + ch);
   }
 }
@@ -316,10 +317,14 @@ SGLC_API int sglc_conv_silu(const float* x, long long x_stride, const float* tap
   const bool vec = C % 4 == 0 && x_stride % 4 == 0 && y_stride % 4 == 0 && al(x) && al(taps) && al(bias) && al(tail) && al(y);
   const int cb = (C + (vec ? 512 : 128) - 1) / (vec ? 512 : 128);
   if (cb + 1 > 65535) return SGLC_ERR_UNSUPPORTED;
-  // tokens a thread: as many as still leave every SM several blocks, up to 8
-  while (p.per < 8 && (long long)((T + 2 * p.per - 1) / (2 * p.per)) * cb >= 148LL * 4) p.per *= 2;
+  // tokens a thread: several where that still leaves every SM several blocks
+  if ((long long)((T + CONV_PER - 1) / CONV_PER) * cb >= 148LL * 4) p.per = CONV_PER;
   const dim3 grid((T + p.per - 1) / p.per, cb + (heads > 0 ? 1 : 0));
-#define GO(CW, KT) return sglc_launch(conv_silu_kernel<CW, KT>, grid, dim3(128), 0, stream, 1, true, p)
+#define GO(CW, KT)                                                                                                    \
+  do {                                                                                                                \
+    if (p.per > 1) return sglc_launch(conv_silu_kernel<CW, KT, CONV_PER>, grid, dim3(128), 0, stream, 1, true, p);    \
+    return sglc_launch(conv_silu_kernel<CW, KT, 1>, grid, dim3(128), 0, stream, 1, true, p);                          \
+  } while (0)
 #define PICK(CW)        \
   switch (K) {          \
     case 1: GO(CW, 1);  \

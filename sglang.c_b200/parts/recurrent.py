@@ -473,8 +473,10 @@ class SelectiveStateSpace(Part):
                       ctx.q_start, ctx.state_slots, ctx.R, gates=(H, C, self.A_log, self.dt_bias, gates))
         y = ctx.alloc((T, inner), torch.float32)
         qkv = ctx.columns(u, inner + G * N, C), ctx.columns(u, inner, inner + G * N), ctx.columns(u, 0, inner)
-        # long portions in chunks side by side, everything else token by token
-        if ops.state_chunks_pay(T, ctx.R, ctx.max_q_len):
+        # one token a request: a pass over the states; long portions: in chunks side by side; else token by token
+        if ctx.max_q_len == 1:
+            ops.state_step(*qkv, gates, y, state.tensor, ctx.state_slots, H, G, N, V, skip=self.D)
+        elif ops.state_chunks_pay(T, ctx.R, ctx.max_q_len):
             inner_mark = ctx.mark()
             ws = ctx.alloc((ops.state_chunks_workspace(T, ctx.R, H, G, N, V),), torch.float32)
             ops.state_chunks(*qkv, gates, self.A_log, y, state.tensor, ctx.q_start, ctx.state_slots, ctx.R, H, G, N, V, ws,

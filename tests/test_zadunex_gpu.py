@@ -146,11 +146,11 @@ def _space_case(rng, n, H, G, N, V):
     return x, B, C, dt
 
 
-@pytest.mark.parametrize("form", ["tokens", "chunks"])
+@pytest.mark.parametrize("form", ["tokens", "chunks", "single"])
 @pytest.mark.parametrize("H,G,N,V", [(4, 2, 24, 20), (3, 1, 7, 5), (2, 2, 128, 64), (2, 1, 160, 72), (6, 3, 64, 64), (1, 1, 256, 130),
                                      (8, 1, 16, 128)])
 def test_state_space_in_portions_by_tokens_and_by_chunks(form, H, G, N, V):
-    """Both forms of the recurrence: three requests of unequal lengths in shuffled slots, whole and in portions
+    """The forms of the recurrence (and the one for single tokens behind the others): three requests of unequal lengths in shuffled slots, whole and in portions
     (down to one token, across chunks' borders), states carried through their slots; the first token,
     which is large, still shows at the end."""
     from sglang_c_b200.csrc import ops
@@ -164,7 +164,7 @@ def test_state_space_in_portions_by_tokens_and_by_chunks(form, H, G, N, V):
     assert np.abs(lost[-1] - want[0][0][-1]).max() > 1e-2 * np.abs(want[0][0]).std()
     flat = [[c[0].reshape(n, -1) for c, n in zip(cases, lens)], [c[1].reshape(n, -1) for c, n in zip(cases, lens)],
             [c[2].reshape(n, -1) for c, n in zip(cases, lens)], [c[3] for c in cases]]
-    for sizes in ((400,), (64, 128, 65), (63, 2, 1, 129)):
+    for sizes in ((400,), (64, 128, 65), (63, 2, 1, 129)) if form != "single" else ((298, 1, 1, 1, 64, 1),):
         state = torch.zeros((6, H, N, V), device=DEV)
         state[[0, 1, 3]] = 7.0
         for step in cuts(lens, sizes):
@@ -173,7 +173,9 @@ def test_state_space_in_portions_by_tokens_and_by_chunks(form, H, G, N, V):
             T, R = xs.shape[0], len(step)
             gates = torch.cat([dts, torch.exp(-torch.exp(dev(A_log)) * dts)], 1).contiguous()
             out = torch.zeros((T, H * V), device=DEV)
-            if form == "tokens":
+            if T == R and form == "single":
+                ops.state_step(Cs, Bs, xs, gates, out, state, sl, H, G, N, V, skip=dev(D))
+            elif form != "chunks":
                 ops.matrix_state("gated", Cs, Bs, xs, out, state, qs, sl, R, H, G, N, V, gates=gates, skip=dev(D))
             else:
                 ws = torch.full((ops.state_chunks_workspace(T, R, H, G, N, V),), float("nan"), device=DEV)
