@@ -15,6 +15,7 @@
 SGLC_DEFINE_ERROR_STRING()
 
 constexpr int STREAMS_MAX = 32;
+constexpr int STREAM_THREADS = 256;
 
 struct StreamArgs {
   const float* src; long long src_row, src_stream;   // old rows: element strides between tokens and streams
@@ -55,7 +56,8 @@ __device__ __forceinline__ float4 normed(const float4& v, float inv, const float
 
 // NS streams are kept in registers; EXACT: there are NS of them, else at most so many.  TV: float or float4.
 template <int NS, bool EXACT, typename TV, typename TO>
-__global__ void stream_step_kernel(const StreamArgs p, TO* __restrict__ h) {
+__global__ void __launch_bounds__(STREAM_THREADS, NS <= 4 ? 4 : 1)
+stream_step_kernel(const StreamArgs p, TO* __restrict__ h) {
   extern __shared__ __align__(16) float srow[];      // u of this row
   __shared__ float red[33];
   __shared__ float wm[STREAMS_MAX * STREAMS_MAX], wo[STREAMS_MAX], wi[STREAMS_MAX];
@@ -87,7 +89,7 @@ __global__ void stream_step_kernel(const StreamArgs p, TO* __restrict__ h) {
     TV u;
     if (yr) {
       const TV yv = yr[i];
-#pragma unroll
+#pragma unroll(NS <= 8 ? NS : 1)
       for (int t = 0; t < NS; t++) {
         if (EXACT || t < S) {
           TV a = times(wo[t], yv);
@@ -158,7 +160,7 @@ SGLC_API int sglc_stream_step(const float* src, long long src_row, long long src
                    al(dst, 16) && al(y, 16) && al(gain, 16) && al(h, h_dtype == SGLC_F32 ? 16 : 8);
   const int work = vec ? E / 4 : E;
   int threads = (work + 31) / 32 * 32;
-  if (threads > 512) threads = 512;
+  if (threads > STREAM_THREADS) threads = STREAM_THREADS;
   if (vec) {
     if (h_dtype == SGLC_BF16) return stream_step_go<float4>(p, (__nv_bfloat16*)h, threads, smem, stream);
     return stream_step_go<float4>(p, (float*)h, threads, smem, stream);
